@@ -5,6 +5,7 @@ from .tefezen import TefezenConfig
 from .zadinex import ZadinexConfig
 from .vuvosun import VuvosunConfig
 from .desalorn import DesalornConfig
+from .pipesun import PipesunConfig
 from .registry import config_from_dict, known_architectures, load_config, register_architecture
 
 register_architecture("Qwen3ForCausalLM", Qwen3Config)
@@ -12,7 +13,8 @@ register_architecture("Tefezen", TefezenConfig)
 register_architecture("Zadinex", ZadinexConfig)
 register_architecture("Vuvosun", VuvosunConfig)
 register_architecture("Desalorn", DesalornConfig)
+register_architecture("Pipesun", PipesunConfig)
 
 __all__ = ["ConfigError", "FeedForwardSpec", "LayerSpec", "MixerSpec", "ModelSpec", "NormSpec",
-           "PositionSpec", "Qwen3Config", "TefezenConfig", "ZadinexConfig", "VuvosunConfig", "DesalornConfig", "config_from_dict", "known_architectures", "load_config",
+           "PositionSpec", "Qwen3Config", "TefezenConfig", "ZadinexConfig", "VuvosunConfig", "DesalornConfig", "PipesunConfig", "config_from_dict", "known_architectures", "load_config",
            "register_architecture"]

@@ -48,7 +48,7 @@ def _lookup(pairs, key, default):
 
 @dataclass(frozen=True)
 class MixerSpec:
-    kind: str                 # "attention" | "latent_attention" | "lightning" | "retention" | "wkv" | "gated_delta" | "mlstm" | "parallel"
+    kind: str                 # "attention" | "latent_attention" | "differential_attention" | "lightning" | "retention" | "wkv" | "gated_delta" | "mlstm" | "parallel"
     hidden_size: int
     num_heads: int = 0
     num_kv_heads: int = 0
@@ -98,7 +98,7 @@ class LayerSpec:
     feed-forward (None), or take more norms than two from ``norms`` (a norm after each part as well as
     before it, say) and its own constants from ``extra``."""
     index: int
-    arrangement: str          # "pre_norm" | "pre_norm_scaled" | "output_norm" | "hyper" | "parallel"
+    arrangement: str          # "pre_norm" | "pre_norm_scaled" | "output_norm" | "hyper" | "parallel" | "sandwich"
     mixer: MixerSpec
     feed_forward: Optional[FeedForwardSpec]
     mixer_norm: Optional[NormSpec]
@@ -188,4 +188,16 @@ def _share_latent(index, me, src, owner):
     return None
 
 
-_SHARING_RULES = {"attention": _share_kv, "latent_attention": _share_latent}
+def _share_pairs(index, me, src, owner):
+    """Differential attention reading another layer's keys and values: the rows hold both maps' keys and the values at the
+    owner's widths, so the head counts and widths must be the same."""
+    for what, a, b in (("key/value heads", me.num_kv_heads, owner.num_kv_heads), ("query heads", me.num_heads, owner.num_heads),
+                       ("heads of", me.head_dim, owner.head_dim), ("values of", me.option("value_dim"), owner.option("value_dim"))):
+        if a != b:
+            return f"layer {index} has {what} {a}, layer {src}, whose cache it reads, has {b}"
+    if owner.position != me.position:
+        return f"layer {index} rotates its keys otherwise than layer {src}, whose cache it reads"
+    return None
+
+
+_SHARING_RULES = {"attention": _share_kv, "latent_attention": _share_latent, "differential_attention": _share_pairs}

@@ -5,7 +5,8 @@
 //                    written after attention)
 //   tb_attn_decode   one query per sequence over its cached keys, cut into splits by the sequence's
 //                    own length (tb_split_keys), each giving (max, sum, unnormalised output)
-//   tb_attn_merge    log-sum-exp merge of the chunks in chunk order (a block per sequence and head)
+//   tb_attn_merge    log-sum-exp merge of the chunks in chunk order (a block per sequence and head, or, with
+//                    AttnArgs.pair_lambda, per sequence and pair of heads, whose difference it finishes)
 //
 // One warp per (query, head): a lane scores one key per round with the whole query in shared
 // memory, the warp folds 32 scores into the running softmax, then every lane accumulates its
@@ -121,7 +122,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_prefill_kernel(AttnArgs a
     extern __shared__ float q_smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x, h = blockIdx.y * ATT_WARPS + warp;
-    if (h >= a.nh) return;
+    if (h >= a.nh) return;                             // (the two heads of a pair leave or stay together)
     const int hd = a.hd;
     float* qs = q_smem + warp * hd;
     load_query<T>(qs, (const T*)a.q + (size_t)t * a.q_stride + h * hd, hd, lane);
@@ -144,6 +145,36 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_prefill_kernel(AttnArgs a
     }
     const float inv = 1.0f / st.l;
     const int hdv = value_width(a);
+    if (a.pair_lambda) {
+        // heads 2p and 2p + 1 sit in neighbouring warps: the second leaves its output where its query lay, and the first
+        // takes it off its own, divides by the root mean square and writes the pair's row
+        if (h & 1) {
+            __syncwarp();
+#pragma unroll
+            for (int j = 0; j < MAXE; ++j) {
+                const int d = lane + 32 * j;
+                if (d < hdv) qs[d] = st.acc[j] * inv;
+            }
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(1 + (warp >> 1)) : "memory");      // the pair's two warps
+        if (h & 1) return;
+        const float lam = *a.pair_lambda;
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < MAXE; ++j) {
+            const int d = lane + 32 * j;
+            st.acc[j] = d < a.pair_width ? fmaf(-lam, qs[hd + d], st.acc[j] * inv) : 0.f;
+            ss = fmaf(st.acc[j], st.acc[j], ss);
+        }
+        const float r = a.pair_scale / sqrtf(warp_sum(ss) / (float)a.pair_width + a.pair_eps);
+        T* o = (T*)a.out + (size_t)t * a.out_stride + (h >> 1) * a.pair_width;
+#pragma unroll
+        for (int j = 0; j < MAXE; ++j) {
+            const int d = lane + 32 * j;
+            if (d < a.pair_width) stf(o + d, st.acc[j] * r);
+        }
+        return;
+    }
     T* o = (T*)a.out + (size_t)t * a.out_stride + h * hdv;
 #pragma unroll
     for (int j = 0; j < MAXE; ++j) {
@@ -197,26 +228,20 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_decode_kernel(AttnArgs a)
     }
 }
 
-// grid (B, nh), one block of up to 128 threads: out = sum_s exp(m_s - m) acc_s / sum_s exp(m_s - m) l_s, splits in
-// order.  Every thread finds the maximum and the weights' sum itself from the splits' (m, l) pairs (a few broadcast
-// loads) and adds up its own output dims, so the loads of different splits do not wait for one another; splits that saw
-// no key (all of them before a window's first key) are skipped.
-template <typename T, int MAXE>
-__global__ void attn_merge_kernel(AttnArgs a) {
-    pdl_launch_dependents();
-    pdl_wait();
-    const int b = blockIdx.x, h = blockIdx.y, hd = value_width(a), stride = hd + 2;
+// The splits of one head in order: acc = sum_s exp(m_s - m) acc_s, returned unnormalised, with l = sum_s exp(m_s - m) l_s
+// (the sink's term included).  Every thread finds the maximum and the weights' sum itself from the splits' (m, l) pairs (a
+// few broadcast loads) and adds up its own output dims, so the loads of different splits do not wait for one another; splits
+// that saw no key (all of them before a window's first key) are skipped.
+template <int PER>
+__device__ __forceinline__ float merge_splits(const AttnArgs& a, int b, int h, int hd, int used, int first, float* acc) {
+    const int stride = hd + 2;
     const float* part = a.scratch + (size_t)(b * a.nh + h) * a.n_splits * stride;
-    const int len = a.batch.kv_len[b], keys = tb_split_keys(len, a.chunk, a.n_splits);
-    const int used = min(a.n_splits, (len + keys - 1) / keys);
-    const int first = (a.window > 0 && a.keep_first <= 0) ? max(0, len - a.window) / keys : 0;      // splits before the window's first key hold nothing
     float m = -FLT_MAX;
     for (int s = first; s < used; ++s)
         if (part[s * stride + hd + 1] > 0.f) m = fmaxf(m, part[s * stride + hd]);
     const bool sunk = a.sink != nullptr;
     if (sunk) m = fmaxf(m, a.sink[h]);
-    constexpr int PER = (32 * MAXE + 127) / 128;
-    float l = 0.f, acc[PER];
+    float l = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; ++j) acc[j] = 0.f;
     for (int s = first; s < used; ++s) {
@@ -232,13 +257,59 @@ __global__ void attn_merge_kernel(AttnArgs a) {
         }
     }
     if (sunk) l += expf(a.sink[h] - m);               // the sink counts once, here, not once a split
-    float inv = 1.0f / l;
+    return l;
+}
+
+// grid (B, nh), one block of up to 128 threads: out = sum_s exp(m_s - m) acc_s / sum_s exp(m_s - m) l_s.
+template <typename T, int MAXE>
+__global__ void attn_merge_kernel(AttnArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int b = blockIdx.x, h = blockIdx.y, hd = value_width(a);
+    const int len = a.batch.kv_len[b], keys = tb_split_keys(len, a.chunk, a.n_splits);
+    const int used = min(a.n_splits, (len + keys - 1) / keys);
+    const int first = (a.window > 0 && a.keep_first <= 0) ? max(0, len - a.window) / keys : 0;      // splits before the window's first key hold nothing
+    constexpr int PER = (32 * MAXE + 127) / 128;
+    float acc[PER];
+    float inv = 1.0f / merge_splits<PER>(a, b, h, hd, used, first, acc);
     if (a.head_gate) inv *= 1.0f / (1.0f + expf(-a.head_gate[(size_t)b * a.head_gate_stride + h]));      // the head's gate
     T* o = (T*)a.out + (size_t)b * a.out_stride + h * hd;
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
         const int d = threadIdx.x + blockDim.x * j;
         if (d < hd) stf(o + d, acc[j] * inv);
+    }
+}
+
+// grid (B, nh / 2), 128 threads: both maps of a pair merged, the second times lambda taken off the first, the difference
+// divided by its root mean square (AttnArgs.pair_lambda).
+template <typename T, int MAXE>
+__global__ void __launch_bounds__(128) attn_merge_pair_kernel(AttnArgs a) {
+    pdl_launch_dependents();
+    pdl_wait();
+    __shared__ float red[33];
+    const int b = blockIdx.x, p = blockIdx.y, hd = value_width(a);
+    const int len = a.batch.kv_len[b], keys = tb_split_keys(len, a.chunk, a.n_splits);
+    const int used = min(a.n_splits, (len + keys - 1) / keys);
+    const int first = (a.window > 0 && a.keep_first <= 0) ? max(0, len - a.window) / keys : 0;
+    constexpr int PER = (32 * MAXE + 127) / 128;
+    float a1[PER], a2[PER];
+    const float inv1 = 1.0f / merge_splits<PER>(a, b, 2 * p, hd, used, first, a1);
+    const float inv2 = 1.0f / merge_splits<PER>(a, b, 2 * p + 1, hd, used, first, a2);
+    const float lam = *a.pair_lambda;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int d = threadIdx.x + blockDim.x * j;
+        a1[j] = d < a.pair_width ? fmaf(-lam, a2[j] * inv2, a1[j] * inv1) : 0.f;
+        ss = fmaf(a1[j], a1[j], ss);
+    }
+    const float r = a.pair_scale / sqrtf(block_sum(ss, red) / (float)a.pair_width + a.pair_eps);
+    T* o = (T*)a.out + (size_t)b * a.out_stride + p * a.pair_width;
+#pragma unroll
+    for (int j = 0; j < PER; ++j) {
+        const int d = threadIdx.x + blockDim.x * j;
+        if (d < a.pair_width) stf(o + d, a1[j] * r);
     }
 }
 
@@ -250,6 +321,10 @@ static int check_common(const AttnArgs& a, const char* who) {
     TB_REQUIRE(a.q_stride % 8 == 0 && a.kv_stride % 8 == 0, "%s: row strides must be multiples of 8 elements", who);
     TB_REQUIRE(a.window >= 0 && a.keep_first >= 0, "%s: negative window or kept tokens", who);
     TB_REQUIRE(!(a.softcap > 0.f) && !a.rel_bias && !a.head_mix, "%s: capped, biased or mixed scores run on the mixed-heads kernels", who);
+    TB_REQUIRE(!a.out_f32, "%s: float32 output rows are the tensor-core prompt kernels'", who);
+    TB_REQUIRE(!a.pair_lambda || (a.nh % 2 == 0 && a.pair_width > 0 && a.pair_width <= value_width(a) && a.pair_eps > 0.f && !a.head_gate && !a.sink),
+               "%s: pairs of heads need an even number of them (%d), a width (%d) within the value's and no gate or sink a head", who, a.nh, a.pair_width);
+    TB_REQUIRE(!a.pair_lambda || value_width(a) <= a.hd, "%s: a pair's value row (%d) may not be wider than its key row (%d)", who, value_width(a), a.hd);
     TB_REQUIRE(!a.cache.storage || (a.cache.head_dim == a.hd && a.cache.kv_heads == a.nkv), "%s: the cache view does not match the heads", who);
     return 0;
 }
@@ -286,9 +361,13 @@ extern "C" int tb_attn_prefill(const AttnArgs* args, int dtype, cudaStream_t str
 extern "C" int tb_attn_merge(const AttnArgs* args, int dtype, cudaStream_t stream) {
     AttnArgs a = *args;
     TB_REQUIRE(dtype == TB_F32 || dtype == TB_BF16, "attn_merge: unknown dtype %d", dtype);
-    dim3 mgrid(a.batch.B, a.nh);
     const bool wide = wide_rows(a);
-    ATT_DISPATCH(attn_merge_kernel, mgrid, 128, 0);
+    if (a.pair_lambda) {
+        TB_REQUIRE(a.nh % 2 == 0 && a.pair_width > 0 && a.pair_width <= value_width(a) && !a.head_gate && !a.sink, "attn_merge: pairs of heads do not fit");
+        ATT_DISPATCH(attn_merge_pair_kernel, dim3(a.batch.B, a.nh / 2), 128, 0);
+    } else {
+        ATT_DISPATCH(attn_merge_kernel, dim3(a.batch.B, a.nh), 128, 0);
+    }
     TB_CHECK_LAUNCH("attn_merge");
     return 0;
 }
@@ -302,11 +381,10 @@ extern "C" int tb_attn_decode(const AttnArgs* args, int dtype, cudaStream_t stre
     TB_REQUIRE(a.nkv <= 65535 && a.head_blocks <= 65535, "attn_decode: too many kv heads");
     TB_REQUIRE(a.head_blocks == 0 || (a.head_blocks > 0 && a.nh % a.head_blocks == 0 && a.head_blocks % a.nkv == 0),
                "attn_decode: %d blocks for %d query heads on %d kv heads", a.head_blocks, a.nh, a.nkv);
-    dim3 grid(a.batch.B, a.head_blocks > 0 ? a.head_blocks : a.nkv, a.n_splits), mgrid(a.batch.B, a.nh);
+    dim3 grid(a.batch.B, a.head_blocks > 0 ? a.head_blocks : a.nkv, a.n_splits);
     const size_t smem = (size_t)ATT_WARPS * a.hd * sizeof(float);
     const bool wide = wide_rows(a);
     ATT_DISPATCH(attn_decode_kernel, grid, ATT_WARPS * 32, smem);
-    ATT_DISPATCH(attn_merge_kernel, mgrid, 128, 0);
     TB_CHECK_LAUNCH("attn_decode");
-    return 0;
+    return tb_attn_merge(args, dtype, stream);
 }

@@ -55,6 +55,16 @@ struct AttnArgs {
     // One gate a (token, head): head_gate[t * head_gate_stride + h] (float32 logits; null: none) multiplies head h's
     // output row by its sigmoid where the softmax is finished (the any-size merge and the mixed-heads kernels).
     const float* head_gate; int head_gate_stride;
+    // Differential attention: query heads 2p and 2p + 1 are two softmax maps over the same values, and what leaves is, a
+    // pair, o = a_2p - *pair_lambda a_2p+1, divided by sqrt(mean(o^2) + pair_eps) over its first pair_width elements (the
+    // rest is padding), times pair_scale: out row [t][p * pair_width ..].  Done where the softmax is finished, in float32:
+    // the any-size prompt kernel and the merge of decode splits (null: no pairs, every head leaves as it is).
+    const float* pair_lambda; float pair_eps; float pair_scale; int pair_width;
+    // The tensor-core prompt kernels: output rows are float32 (a kernel that finishes them in float32 follows).
+    int out_f32;
+    // The tensor-core kernels: softmax weights enter the product with the values as two bfloat16 halves (the rounded weight
+    // and what rounding left over), so that they keep sixteen bits instead of eight.
+    int exact_weights;
 };
 
 // How decode attention cuts the keys of ONE sequence into splits: ``chunk`` keys each while ``n_splits`` of

@@ -479,6 +479,7 @@ int check_mixed(const AttnArgs& a, const char* who) {
     TB_REQUIRE(a.window >= 0 && a.keep_first == 0 && !a.sink, "%s: no kept first tokens and no sink here", who);
     TB_REQUIRE(!a.cache.storage || (a.cache.head_dim == a.hd && a.cache.kv_heads == a.nkv), "%s: the cache view does not match the heads", who);
     TB_REQUIRE(!a.rel_bias || a.rel_far >= 0, "%s: the distance table needs its last row's distance", who);
+    TB_REQUIRE(!a.pair_lambda && !a.out_f32, "%s: pairs of heads run on the other attention kernels", who);
     TB_REQUIRE(!a.head_gate || a.head_gate_stride >= a.nh, "%s: the heads' gates need a row of at least %d", who, a.nh);
     return 0;
 }

@@ -77,6 +77,10 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     const __nv_bfloat162 p = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&p);
 }
+// The two parts of (lo, hi) that rounding them to the pair ``rounded`` left over, themselves rounded.
+__device__ __forceinline__ uint32_t rest2(float lo, float hi, uint32_t rounded) {
+    return pack2(lo - __uint_as_float(rounded << 16), hi - __uint_as_float(rounded & 0xffff0000u));
+}
 // Byte offset of (row, 16-byte chunk of the row's 128 bytes) in a 64-row, 128-byte-swizzled box.
 __device__ __forceinline__ uint32_t swz(int row, int chunk16) { return (uint32_t)(row * 128 + ((chunk16 ^ (row & 7)) << 4)); }
 
@@ -122,7 +126,8 @@ __device__ __forceinline__ void fused_head(float row_scale, bool normed, const f
     }
 }
 
-template <int HD, bool WIDE, bool CL, bool FUSED = false>
+// EXACT: softmax weights enter P . V as two bfloat16 halves (AttnArgs.exact_weights).
+template <int HD, bool WIDE, bool CL, bool FUSED = false, bool EXACT = false>
 __global__ void __launch_bounds__(DEC_THREADS)
 attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kv_map, DecArgs a) {
     static_assert(!FUSED || CL, "the folded head norm needs the cluster's barrier to know when the sums may be cleared");
@@ -378,6 +383,11 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kv_map, DecArgs a) {
         l1 = l1 * al1 + p[0][2] + p[0][3] + p[1][2] + p[1][3];
         const uint32_t pa0 = pack2(p[0][0], p[0][1]), pa1 = pack2(p[0][2], p[0][3]);
         const uint32_t pa2 = pack2(p[1][0], p[1][1]), pa3 = pack2(p[1][2], p[1][3]);
+        uint32_t pb0 = 0, pb1 = 0, pb2 = 0, pb3 = 0;                      // EXACT: what rounding left over
+        if (EXACT) {
+            pb0 = rest2(p[0][0], p[0][1], pa0); pb1 = rest2(p[0][2], p[0][3], pa1);
+            pb2 = rest2(p[1][0], p[1][1], pa2); pb3 = rest2(p[1][2], p[1][3], pa3);
+        }
         // O[16 x HD] = alpha * O + P . V over this warp's 16 keys
         {
             const int mtx = lane >> 3, r = lane & 7;
@@ -391,6 +401,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kv_map, DecArgs a) {
                 o[n + 1][0] *= al0; o[n + 1][1] *= al0; o[n + 1][2] *= al1; o[n + 1][3] *= al1;
                 mma_bf16(o[n], pa0, pa1, pa2, pa3, b0, b1);
                 mma_bf16(o[n + 1], pa0, pa1, pa2, pa3, b2, b3);
+                if (EXACT) { mma_bf16(o[n], pb0, pb1, pb2, pb3, b0, b1); mma_bf16(o[n + 1], pb0, pb1, pb2, pb3, b2, b3); }
             }
         }
         __syncwarp();
@@ -503,7 +514,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kv_map, DecArgs a) {
 // the step's own keys were appended before).  Key tiles of 64 run from the window's first key to the
 // diagonal; S and P.V are mma.sync.m16n8k16 as above.  Heavy (late) query blocks are scheduled first.
 struct PreArgs {
-    __nv_bfloat16* out; int out_stride;
+    void* out; int out_stride; int out_f32;  // bfloat16 rows, or float32 ones
     const int* q_start; int B;
     int nh; int nkv; int window; float scale_log2;
     int k_col0; int v_col0;                  // first column of the K heads and of the V heads
@@ -517,7 +528,8 @@ struct PreArgs {
 // HDK: dimensions of a query and of a key; HDV: of a value and of an output row (the same for grouped-query attention).
 // HDT: the last HDT of a key's HDK dimensions are shared by all heads and come from a third buffer (``tail_map``, at
 // column tail_col0 of the token's row): a key that is [a part of its own head | a rotated part common to all heads].
-template <int HDK, int HDV, int HDT>
+// EXACT: softmax weights enter P . V as two bfloat16 halves (AttnArgs.exact_weights).
+template <int HDK, int HDV, int HDT, bool EXACT>
 __global__ void __launch_bounds__(DEC_THREADS, 2)
 attn_prefill_mma_kernel(const __grid_constant__ CUtensorMap qkv_map, const __grid_constant__ CUtensorMap kv_map,
                         const __grid_constant__ CUtensorMap tail_map, PreArgs a) {
@@ -661,6 +673,11 @@ attn_prefill_mma_kernel(const __grid_constant__ CUtensorMap qkv_map, const __gri
         for (int kk = 0; kk < 4; ++kk) {
             const uint32_t pa0 = pack2(sc[2 * kk][0], sc[2 * kk][1]), pa1 = pack2(sc[2 * kk][2], sc[2 * kk][3]);
             const uint32_t pa2 = pack2(sc[2 * kk + 1][0], sc[2 * kk + 1][1]), pa3 = pack2(sc[2 * kk + 1][2], sc[2 * kk + 1][3]);
+            uint32_t pb0 = 0, pb1 = 0, pb2 = 0, pb3 = 0;
+            if (EXACT) {
+                pb0 = rest2(sc[2 * kk][0], sc[2 * kk][1], pa0); pb1 = rest2(sc[2 * kk][2], sc[2 * kk][3], pa1);
+                pb2 = rest2(sc[2 * kk + 1][0], sc[2 * kk + 1][1], pa2); pb3 = rest2(sc[2 * kk + 1][2], sc[2 * kk + 1][3], pa3);
+            }
             const int key = kk * 16 + (mtx & 1) * 8 + r;
 #pragma unroll
             for (int nn = 0; nn < NT; nn += 2) {
@@ -669,6 +686,7 @@ attn_prefill_mma_kernel(const __grid_constant__ CUtensorMap qkv_map, const __gri
                 ldsm_x4_trans(vs_base + (dim0 >> 6) * 8192 + swz(key, (dim0 & 63) >> 3), b0, b1, b2, b3);
                 mma_bf16(o[nn], pa0, pa1, pa2, pa3, b0, b1);
                 mma_bf16(o[nn + 1], pa0, pa1, pa2, pa3, b2, b3);
+                if (EXACT) { mma_bf16(o[nn], pb0, pb1, pb2, pb3, b0, b1); mma_bf16(o[nn + 1], pb0, pb1, pb2, pb3, b2, b3); }
             }
         }
         __syncwarp();
@@ -677,8 +695,19 @@ attn_prefill_mma_kernel(const __grid_constant__ CUtensorMap qkv_map, const __gri
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
     const float i0 = a.sink ? sink_factor(a.sink, h, m0, l0) : 1.0f / l0, i1 = a.sink ? sink_factor(a.sink, h, m1, l1) : 1.0f / l1;
-    __nv_bfloat16* out0 = a.out + (size_t)(tok0 + qr0) * a.out_stride + h * HDV + 2 * t;
-    __nv_bfloat16* out1 = a.out + (size_t)(tok0 + qr1) * a.out_stride + h * HDV + 2 * t;
+    const size_t at0 = (size_t)(tok0 + qr0) * a.out_stride + h * HDV + 2 * t, at1 = (size_t)(tok0 + qr1) * a.out_stride + h * HDV + 2 * t;
+    if (a.out_f32) {
+        float* f0 = (float*)a.out + at0;
+        float* f1 = (float*)a.out + at1;
+#pragma unroll
+        for (int nn = 0; nn < NT; ++nn) {
+            if (qr0 < n) *reinterpret_cast<float2*>(f0 + nn * 8) = make_float2(o[nn][0] * i0, o[nn][1] * i0);
+            if (qr1 < n) *reinterpret_cast<float2*>(f1 + nn * 8) = make_float2(o[nn][2] * i1, o[nn][3] * i1);
+        }
+        return;
+    }
+    __nv_bfloat16* out0 = (__nv_bfloat16*)a.out + at0;
+    __nv_bfloat16* out1 = (__nv_bfloat16*)a.out + at1;
 #pragma unroll
     for (int nn = 0; nn < NT; ++nn) {
         if (qr0 < n) *reinterpret_cast<uint32_t*>(out0 + nn * 8) = pack2(o[nn][0] * i0, o[nn][1] * i0);
@@ -696,22 +725,22 @@ template <int HD> constexpr size_t decode_smem() {
     return 1024 + (size_t)(HD == 128 ? 3 : 4) * 2 * PAGE * HD * 2 + 2 * (HD == 128 ? 3 : 4) * sizeof(uint64_t) + 16 + 16 * HD * 2 +
            (16 * HD + 16 + 16 * 32) * sizeof(float);      // the parts received for the merge: up to 16 splits x (share + 32)
 }
-template <int HD, bool WIDE, bool CL, bool FUSED = false>
+template <int HD, bool WIDE, bool CL, bool FUSED = false, bool EXACT = false>
 static int launch_decode(const CUtensorMap& map, const DecArgs& d, dim3 grid, cudaStream_t stream) {
     constexpr size_t smem = decode_smem<HD>();
     static bool configured = false;
     if (!configured) {
-        const cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);   // room for several CTAs per SM
-        if (CL) cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);    // clusters of up to 16
+        const cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED, EXACT>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);   // room for several CTAs per SM
+        if (CL) cudaFuncSetAttribute(attn_decode_mma_kernel<HD, WIDE, CL, FUSED, EXACT>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);    // clusters of up to 16
         TB_REQUIRE(e == cudaSuccess, "attn_decode_mma: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
     if (CL) {
-        const cudaError_t e = tb_launch_cluster_z(attn_decode_mma_kernel<HD, WIDE, CL, FUSED>, grid, DEC_THREADS, smem, stream, (int)grid.z, map, d);
+        const cudaError_t e = tb_launch_cluster_z(attn_decode_mma_kernel<HD, WIDE, CL, FUSED, EXACT>, grid, DEC_THREADS, smem, stream, (int)grid.z, map, d);
         TB_REQUIRE(e == cudaSuccess, "attn_decode_mma: cluster launch failed: %s", cudaGetErrorString(e));
     } else {
-        tb_launch(attn_decode_mma_kernel<HD, WIDE, CL, FUSED>, grid, DEC_THREADS, smem, stream, map, d);
+        tb_launch(attn_decode_mma_kernel<HD, WIDE, CL, FUSED, EXACT>, grid, DEC_THREADS, smem, stream, map, d);
     }
     return 0;
 }
@@ -742,7 +771,12 @@ static int cluster_limit() {
 }
 // Launches the kernel; *merged says whether the splits merged among themselves (a cluster) or left their parts in scratch.
 template <int HD, bool WIDE>
-static int launch_decode_any(const CUtensorMap& map, const DecArgs& d, dim3 grid, bool may_cluster, bool* merged, cudaStream_t stream) {
+static int launch_decode_any(const CUtensorMap& map, const DecArgs& d, dim3 grid, bool may_cluster, bool exact, bool* merged, cudaStream_t stream) {
+    if (exact) {                     // parts in scratch: the merge kernel finishes
+        *merged = false;
+        TB_REQUIRE(d.scratch && !d.acc, "attn_decode_mma: exact weights leave their parts in scratch memory");
+        return launch_decode<HD, WIDE, false, false, true>(map, d, grid, stream);
+    }
     *merged = may_cluster && (int)grid.z <= cluster_limit<HD, WIDE>();
     if (d.acc) {
         TB_REQUIRE(*merged, "attn_decode_mma: the folded head norm needs the splits to form a cluster (%d splits)", (int)grid.z);
@@ -770,6 +804,8 @@ extern "C" int tb_attn_decode_mma_check(const AttnArgs* a, int dtype) {
     TB_REQUIRE(!a->v_alias && (a->hd_v == 0 || a->hd_v == a->hd), "tensor-core attention: keys and values of one width, stored apart");
     TB_REQUIRE(a->cache.page_size == PAGE, "attn_decode_mma: pages of %d rows, not %d", PAGE, a->cache.page_size);
     TB_REQUIRE(a->nkv > 0 && a->nh % a->nkv == 0 && a->nh / a->nkv <= 16, "attn_decode_mma: at most 16 query heads per kv head");
+    TB_REQUIRE(!a->out_f32 && !((a->pair_lambda || a->exact_weights) && a->fused_qk), "attn_decode_mma: pairs of heads and exact weights come with the head norm as a kernel of its own");
+    TB_REQUIRE(!a->pair_lambda || (a->nh % 2 == 0 && a->pair_width > 0 && a->pair_width <= a->hd && !a->sink), "attn_decode_mma: pairs of heads do not fit");
     TB_REQUIRE(a->chunk > 0 && a->chunk % PAGE == 0, "attn_decode_mma: the chunk %d must be a multiple of %d", a->chunk, PAGE);
     if (a->fused_qk) {
         const QkArgs& q = *a->fused_qk;
@@ -793,7 +829,7 @@ extern "C" int tb_attn_decode_mma(const AttnArgs* args, cudaStream_t stream) {
     const AttnArgs& a = *args;
     if (tb_attn_decode_mma_check(args, TB_BF16)) return 1;
     // few enough splits form a cluster and merge among themselves; more leave parts in scratch and tb_attn_merge finishes
-    const bool may_cluster = g_decode_cluster && a.out != nullptr;
+    const bool may_cluster = g_decode_cluster && a.out != nullptr && !a.pair_lambda, exact = a.exact_weights != 0;
     TB_REQUIRE(a.batch.B > 0 && a.cache.storage, "attn_decode_mma: needs sequences and a cache");
     TB_REQUIRE(a.n_splits > 0 && a.n_splits <= 65535 && a.nkv <= 65535, "attn_decode_mma: bad grid");
     TB_REQUIRE(a.cache.head_dim == a.hd && a.cache.kv_heads == a.nkv, "attn_decode_mma: the cache view does not match the heads");
@@ -822,8 +858,8 @@ extern "C" int tb_attn_decode_mma(const AttnArgs* args, cudaStream_t stream) {
     const bool wide = a.nh / a.nkv > 8;
     int rc;
     bool merged = false;
-    if (a.hd == 128) rc = wide ? launch_decode_any<128, true>(map, d, grid, may_cluster, &merged, stream) : launch_decode_any<128, false>(map, d, grid, may_cluster, &merged, stream);
-    else rc = wide ? launch_decode_any<64, true>(map, d, grid, may_cluster, &merged, stream) : launch_decode_any<64, false>(map, d, grid, may_cluster, &merged, stream);
+    if (a.hd == 128) rc = wide ? launch_decode_any<128, true>(map, d, grid, may_cluster, exact, &merged, stream) : launch_decode_any<128, false>(map, d, grid, may_cluster, exact, &merged, stream);
+    else rc = wide ? launch_decode_any<64, true>(map, d, grid, may_cluster, exact, &merged, stream) : launch_decode_any<64, false>(map, d, grid, may_cluster, exact, &merged, stream);
     if (rc) return rc;
     TB_CHECK_LAUNCH("attn_decode_mma");
     return merged ? 0 : tb_attn_merge(args, TB_BF16, stream);
@@ -837,18 +873,24 @@ extern "C" int tb_attn_mma_error() {
     return (int)v;
 }
 
-template <int HDK, int HDV = HDK, int HDT = 0>
-static int launch_prefill(const CUtensorMap& map, const CUtensorMap& kv_map, const CUtensorMap& tail_map, const PreArgs& p, dim3 grid, cudaStream_t stream) {
+template <int HDK, int HDV, int HDT, bool EXACT>
+static int launch_prefill_as(const CUtensorMap& map, const CUtensorMap& kv_map, const CUtensorMap& tail_map, const PreArgs& p, dim3 grid, cudaStream_t stream) {
     constexpr size_t smem = 1024 + (size_t)(2 * (HDK + HDV) + HDK) * 64 * 2 + 8 * sizeof(uint64_t);
     static bool configured = false;
     if (!configured) {
-        const cudaError_t e = cudaFuncSetAttribute(attn_prefill_mma_kernel<HDK, HDV, HDT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        cudaFuncSetAttribute(attn_prefill_mma_kernel<HDK, HDV, HDT>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);   // room for several CTAs per SM
+        const cudaError_t e = cudaFuncSetAttribute(attn_prefill_mma_kernel<HDK, HDV, HDT, EXACT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        cudaFuncSetAttribute(attn_prefill_mma_kernel<HDK, HDV, HDT, EXACT>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);   // room for several CTAs per SM
         TB_REQUIRE(e == cudaSuccess, "attn_prefill_mma: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
         configured = true;
     }
-    tb_launch(attn_prefill_mma_kernel<HDK, HDV, HDT>, grid, DEC_THREADS, smem, stream, map, kv_map, tail_map, p);
+    tb_launch(attn_prefill_mma_kernel<HDK, HDV, HDT, EXACT>, grid, DEC_THREADS, smem, stream, map, kv_map, tail_map, p);
     return 0;
+}
+
+template <int HDK, int HDV = HDK, int HDT = 0>
+static int launch_prefill(const CUtensorMap& map, const CUtensorMap& kv_map, const CUtensorMap& tail_map, const PreArgs& p, bool exact, dim3 grid, cudaStream_t stream) {
+    return exact ? launch_prefill_as<HDK, HDV, HDT, true>(map, kv_map, tail_map, p, grid, stream)
+                 : launch_prefill_as<HDK, HDV, HDT, false>(map, kv_map, tail_map, p, grid, stream);
 }
 
 // 0 if the tensor-core prompt kernel takes this problem, else 1 with the reason.  source: TB_KV_FROM_STEP (every
@@ -871,6 +913,8 @@ extern "C" int tb_attn_prefill_mma_check(const AttnArgs* a, int dtype, int sourc
         TB_REQUIRE(a->cache.storage && a->cache.page_size == PAGE && a->cache.ring_rows == 0, "attn_prefill_mma: needs a cache of %d-row pages that keeps every key", PAGE);
         TB_REQUIRE(a->cache.head_dim == a->hd && a->cache.kv_heads == a->nkv, "attn_prefill_mma: the cache view does not match the heads");
     }
+    TB_REQUIRE(!a->pair_lambda, "attn_prefill_mma: pairs of heads are finished by a kernel of its own behind this one (out_f32)");
+    TB_REQUIRE(!a->out_f32 || (((uintptr_t)a->out & 7) == 0), "attn_prefill_mma: float32 output must be 8-byte aligned");
     TB_REQUIRE(a->out_stride % 2 == 0 && ((uintptr_t)a->out & 3) == 0, "attn_prefill_mma: the output must be 4-byte aligned");
     return 0;
 }
@@ -887,14 +931,15 @@ extern "C" int tb_attn_prefill_mma(const AttnArgs* args, int source, cudaStream_
     if (p.paged && tb_make_map_bf16(&kv_map, a.cache.storage, 2LL * a.cache.num_pages * a.nkv * PAGE, a.hd, a.hd, PAGE)) return 1;
     p.start_pos = a.batch.start_pos; p.slot_of_seq = a.batch.slot_of_seq; p.table = a.cache.table; p.table_width = a.cache.table_width;
     p.v_row0 = a.cache.num_pages * a.nkv * PAGE;
-    p.out = (__nv_bfloat16*)a.out; p.out_stride = a.out_stride; p.q_start = a.batch.q_start; p.B = a.batch.B;
+    p.out = a.out; p.out_stride = a.out_stride; p.out_f32 = a.out_f32; p.q_start = a.batch.q_start; p.B = a.batch.B;
     p.nh = a.nh; p.nkv = a.nkv; p.window = a.window; p.scale_log2 = a.scale * 1.4426950408889634f;
     p.k_col0 = a.nh * a.hd; p.v_col0 = (a.nh + a.nkv) * a.hd; p.tail_col0 = 0; p.sink = a.sink;
     p.keep_first = a.window > 0 ? a.keep_first : 0;
     const int blocks = (a.batch.T + 63) / 64 + a.batch.B;          // upper bound on sum over sequences of ceil(n / 64)
     TB_REQUIRE(blocks <= 65535, "attn_prefill_mma: too many query blocks (%d)", blocks);
     dim3 grid(a.nh, blocks);
-    const int rc = a.hd == 128 ? launch_prefill<128>(map, kv_map, kv_map, p, grid, stream) : launch_prefill<64>(map, kv_map, kv_map, p, grid, stream);
+    const bool exact = a.exact_weights != 0;
+    const int rc = a.hd == 128 ? launch_prefill<128>(map, kv_map, kv_map, p, exact, grid, stream) : launch_prefill<64>(map, kv_map, kv_map, p, exact, grid, stream);
     if (rc) return rc;
     TB_CHECK_LAUNCH("attn_prefill_mma");
     return 0;
@@ -913,6 +958,8 @@ struct SplitAttnArgs {
     void* out; int out_stride;
     TbBatch batch;
     int nh; int dn; int dt; int dv; int window; float scale;
+    const float* sink;                       // [nh] or null: one more term exp(sink) of every head's softmax denominator
+    int exact_weights;                       // softmax weights enter the product with the values as two bfloat16 halves
 };
 
 extern "C" int tb_attn_prefill_split_check(const SplitAttnArgs* a) {
@@ -936,13 +983,13 @@ extern "C" int tb_attn_prefill_split(const SplitAttnArgs* args, cudaStream_t str
     if (tb_make_map_bf16(&tail_map, a.tail, a.batch.T, a.tail_stride, a.tail_stride, 64)) return 1;
     PreArgs p;
     p.paged = 0; p.start_pos = nullptr; p.slot_of_seq = nullptr; p.table = nullptr; p.table_width = 0; p.v_row0 = 0;
-    p.out = (__nv_bfloat16*)a.out; p.out_stride = a.out_stride; p.q_start = a.batch.q_start; p.B = a.batch.B;
+    p.out = a.out; p.out_stride = a.out_stride; p.out_f32 = 0; p.q_start = a.batch.q_start; p.B = a.batch.B;
     p.nh = a.nh; p.nkv = a.nh; p.window = a.window; p.scale_log2 = a.scale * 1.4426950408889634f;
-    p.k_col0 = a.k_col0; p.v_col0 = a.v_col0; p.tail_col0 = a.tail_col0; p.sink = nullptr; p.keep_first = 0;
+    p.k_col0 = a.k_col0; p.v_col0 = a.v_col0; p.tail_col0 = a.tail_col0; p.sink = a.sink; p.keep_first = 0;
     const int blocks = (a.batch.T + 63) / 64 + a.batch.B;
     TB_REQUIRE(blocks <= 65535, "attn_prefill_split: too many query blocks (%d)", blocks);
     dim3 grid(a.nh, blocks);
-    const int rc = launch_prefill<192, 128, 64>(q_map, kv_map, tail_map, p, grid, stream);
+    const int rc = launch_prefill<192, 128, 64>(q_map, kv_map, tail_map, p, a.exact_weights != 0, grid, stream);
     if (rc) return rc;
     TB_CHECK_LAUNCH("attn_prefill_split");
     return 0;

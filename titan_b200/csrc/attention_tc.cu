@@ -54,7 +54,7 @@ constexpr uint32_t KV_BOX = BKEY * 128;
 constexpr int KV_STAGES = 4;                           // K and V tiles in flight: the loads run well ahead of P.V
 
 struct TcAttnArgs {
-    __nv_bfloat16* out; int out_stride;
+    void* out; int out_stride; int out_f32;      // bfloat16 rows, or float32 ones
     const int* q_start; int B;
     int nh; int nkv; int window; float scale_log2;
     int keep_first;          // with a window: a sequence's first keep_first keys stay visible to every later query
@@ -119,6 +119,9 @@ constexpr float RESCALE_LOG2 = 8.0f;
 //                          arrives (and before a rescale, and once after its last tile); P.V_{j+4} needs
 //                          all three to have moved on.
 
+// EXACT: the softmax weights enter P . V as two bfloat16 halves (AttnArgs.exact_weights): the rounded weights over the first
+// half of the tile's S columns, what rounding left over over the second half, and each value tile is multiplied by both.
+template <bool EXACT>
 __global__ void __launch_bounds__(THREADS, 1)
 attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_constant__ CUtensorMap kv_map, TcAttnArgs a) {
     extern __shared__ uint8_t smem_raw[];
@@ -243,6 +246,11 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_c
 #pragma unroll
                 for (int ks = 0; ks < BKEY / 16; ++ks)      // 16 keys per step: 8 columns of P, 16 rows of V
                     tc_mma_a_tmem(d, p_tmem + ks * 8, v_desc + (uint64_t)((ks * 2048) >> 4), IDESC_PV, (j >= 2 || ks > 0) ? 1u : 0u);
+                if (EXACT) {
+#pragma unroll
+                    for (int ks = 0; ks < BKEY / 16; ++ks)
+                        tc_mma_a_tmem(d, p_tmem + BKEY / 2 + ks * 8, v_desc + (uint64_t)((ks * 2048) >> 4), IDESC_PV, 1u);
+                }
                 tc_commit(pv_done + (j & 3));               // one arrival for the V ring, the S issuer and the group
             }
         }
@@ -310,6 +318,12 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_c
 #pragma unroll
             for (int i = 0; i < 32; ++i) pk[i] = pack_bf16x2(v[2 * i], v[2 * i + 1]);
             tmem_st32_bits(tmem_s + (j & 3) * BKEY + lane_addr, pk);
+            if (EXACT) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i)
+                    pk[i] = pack_bf16x2(v[2 * i] - __uint_as_float(pk[i] << 16), v[2 * i + 1] - __uint_as_float(pk[i] & 0xffff0000u));
+                tmem_st32_bits(tmem_s + (j & 3) * BKEY + lane_addr + BKEY / 2, pk);
+            }
             // The P.V issuer must have seen this group's previous arrival before the next one, or the
             // barrier would run two phases ahead of it and its parity wait would never end.  P.V of that
             // tile complete implies it; by now (a whole tile later) this wait is almost always over.
@@ -346,12 +360,19 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_c
         if (n_tiles > 1) tmem_wait_ld<64>(o1);
         if (r0 + row < n) {
             const float c0 = w0 * inv, c1 = w1 * inv;
-            __nv_bfloat16* dst = a.out + (size_t)(tok0 + r0 + row) * a.out_stride + h * HD + g * 64;
+            const size_t at = (size_t)(tok0 + r0 + row) * a.out_stride + h * HD + g * 64;
+            __nv_bfloat16* dst = (__nv_bfloat16*)a.out + at;
+            float* dst32 = (float*)a.out + at;
 #pragma unroll
             for (int i = 0; i < 64; i += 8) {
                 float r[8];
 #pragma unroll
                 for (int e = 0; e < 8; ++e) r[e] = n_tiles > 1 ? o0[i + e] * c0 + o1[i + e] * c1 : o0[i + e] * c0;
+                if (a.out_f32) {
+                    *reinterpret_cast<float4*>(dst32 + i) = make_float4(r[0], r[1], r[2], r[3]);
+                    *reinterpret_cast<float4*>(dst32 + i + 4) = make_float4(r[4], r[5], r[6], r[7]);
+                    continue;
+                }
                 uint4 pk;
                 pk.x = pack_bf16x2(r[0], r[1]); pk.y = pack_bf16x2(r[2], r[3]);
                 pk.z = pack_bf16x2(r[4], r[5]); pk.w = pack_bf16x2(r[6], r[7]);
@@ -375,6 +396,7 @@ attn_prefill_tc_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_c
 // that keeps every key: no ring).
 extern "C" int tb_attn_prefill_tc_check(const AttnArgs* a, int dtype, int source) {
     TB_REQUIRE(!(a->softcap > 0.f) && !a->rel_bias && !a->head_mix && !a->head_gate, "attn_prefill_tc: capped, biased, mixed or gated scores run on the mixed-heads kernels");
+    TB_REQUIRE(!a->pair_lambda, "attn_prefill_tc: pairs of heads are finished by a kernel of its own behind this one (out_f32)");
     TB_REQUIRE(a->keep_first >= 0, "attn_prefill_tc: a negative count of kept tokens");
     TB_REQUIRE(dtype == TB_BF16, "attn_prefill_tc: bfloat16 only");
     TB_REQUIRE(source == TB_KV_FROM_STEP || source == TB_KV_FROM_CACHE, "attn_prefill_tc: a sequence continues from the cache and its keys are not all there");
@@ -408,21 +430,22 @@ extern "C" int tb_attn_prefill_tc(const AttnArgs* args, int source, cudaStream_t
     } else if (tb_make_map_bf16(&kv_map, a.q, a.batch.T, a.q_stride, a.q_stride, BKEY)) return 1;
     p.start_pos = a.batch.start_pos; p.slot_of_seq = a.batch.slot_of_seq; p.table = a.cache.table; p.table_width = a.cache.table_width;
     p.v_row0 = a.cache.num_pages * a.nkv * BKEY;
-    p.out = (__nv_bfloat16*)a.out; p.out_stride = a.out_stride; p.q_start = a.batch.q_start; p.B = a.batch.B;
+    p.out = a.out; p.out_stride = a.out_stride; p.out_f32 = a.out_f32; p.q_start = a.batch.q_start; p.B = a.batch.B;
     p.nh = a.nh; p.nkv = a.nkv; p.window = a.window; p.scale_log2 = a.scale * 1.4426950408889634f; p.sink = a.sink;
     p.keep_first = a.window > 0 ? a.keep_first : 0;
     p.k_col0 = a.nh * a.hd; p.v_col0 = (a.nh + a.nkv) * a.hd;
     constexpr size_t smem = 1024 + Q_BYTES + KV_STAGES * 2 * KV_TILE + 256 + 4 * 128 * sizeof(float);
     static_assert(KV_STAGES == 4, "the second kernel's barrier layout and S buffers assume four stages");
-    static bool configured = false;
-    if (!configured) {
-        const cudaError_t e = cudaFuncSetAttribute(attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    auto kernel = a.exact_weights ? attn_prefill_tc_kernel<true> : attn_prefill_tc_kernel<false>;
+    static bool configured[2] = {false, false};
+    if (!configured[a.exact_weights != 0]) {
+        const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         TB_REQUIRE(e == cudaSuccess, "attn_prefill_tc: cannot reserve %zu bytes of shared memory: %s", smem, cudaGetErrorString(e));
-        configured = true;
+        configured[a.exact_weights != 0] = true;
     }
     const int blocks = (a.batch.T + BQ - 1) / BQ + a.batch.B;      // upper bound on sum over sequences of ceil(n / 128)
     TB_REQUIRE(blocks <= 65535, "attn_prefill_tc: too many query blocks (%d)", blocks);
-    tb_launch(attn_prefill_tc_kernel, dim3(a.nh, blocks), THREADS, smem, stream, q_map, kv_map, p);      // heads fastest: the heaviest blocks of all heads start first
+    tb_launch(kernel, dim3(a.nh, blocks), THREADS, smem, stream, q_map, kv_map, p);      // heads fastest: the heaviest blocks of all heads start first
     TB_CHECK_LAUNCH("attn_prefill_tc");
     return 0;
 }

@@ -5,7 +5,8 @@
 //                  activation of a feed-forward without a gate.  The three sums of squares and the result are float32;
 //                  z is read in the compute dtype and y written in it.  One block a row.
 //   tb_gate_rows   y = x * act(g) * scale, element by element over rows (act: sigmoid or silu in float32): the output gate
-//                  of an attention mixer, with the factor of a mixer that runs beside another.  In place if y == x.
+//                  of an attention mixer, with the factor of a mixer that runs beside another.  In place if y == x; g may be float32
+//                  beside rows in bfloat16 (tb_gate_rows_from).
 //   tb_head_norm_gate   per head of dv elements: y = o / sqrt(mean(o^2) + eps) * w * act(g) * scale, o float32, the weight
 //                  one row of dv for all heads or a row per head.  One warp a (token, head).
 #include "common.cuh"
@@ -39,8 +40,8 @@ __global__ void __launch_bounds__(256) polynorm_kernel(const T* z, int ldz, cons
     }
 }
 
-template <typename T>
-__global__ void __launch_bounds__(256) gate_rows_kernel(const T* x, int ldx, const T* __restrict__ g, int ldg,
+template <typename T, typename G>
+__global__ void __launch_bounds__(256) gate_rows_kernel(const T* x, int ldx, const G* __restrict__ g, int ldg,
                                                         T* y, int ldy, int n, int act, float scale) {
     pdl_launch_dependents();
     pdl_wait();
@@ -78,23 +79,31 @@ extern "C" int tb_polynorm(const void* z, int ldz, const float* coef, float eps,
     return 0;
 }
 
-extern "C" int tb_gate_rows(const void* x, int ldx, const void* g, int ldg, void* y, int ldy, int dtype, int rows, int n, int act, float scale,
-                            cudaStream_t stream) {
-    TB_REQUIRE(x && g && y && rows > 0 && n > 0 && rows <= 65535 * 32, "gate_rows: rows are wanted (rows=%d n=%d)", rows, n);
-    TB_REQUIRE(act == 0 || act == 1, "gate_rows: the gate is a sigmoid (0) or silu (1)");
+template <typename T, typename G>
+static void launch_gate_rows(const void* x, int ldx, const void* g, int ldg, void* y, int ldy, int rows, int n, int act, float scale, cudaStream_t stream) {
     for (int r0 = 0; r0 < rows; r0 += 65535) {
         const int nr = rows - r0 < 65535 ? rows - r0 : 65535;
-        dim3 grid((n + 255) / 256, nr);
-        if (dtype == TB_F32)
-            tb_launch(gate_rows_kernel<float>, grid, dim3(256), 0, stream, (const float*)x + (size_t)r0 * ldx, ldx, (const float*)g + (size_t)r0 * ldg, ldg,
-                      (float*)y + (size_t)r0 * ldy, ldy, n, act, scale);
-        else if (dtype == TB_BF16)
-            tb_launch(gate_rows_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)x + (size_t)r0 * ldx, ldx,
-                      (const __nv_bfloat16*)g + (size_t)r0 * ldg, ldg, (__nv_bfloat16*)y + (size_t)r0 * ldy, ldy, n, act, scale);
-        else TB_REQUIRE(false, "gate_rows: unknown dtype %d", dtype);
+        tb_launch(gate_rows_kernel<T, G>, dim3((n + 255) / 256, nr), dim3(256), 0, stream, (const T*)x + (size_t)r0 * ldx, ldx, (const G*)g + (size_t)r0 * ldg, ldg,
+                  (T*)y + (size_t)r0 * ldy, ldy, n, act, scale);
     }
+}
+
+// The gate's rows in a dtype of their own (g_dtype): float32 gate logits that came out of one product with other projections.
+extern "C" int tb_gate_rows_from(const void* x, int ldx, const void* g, int ldg, int g_dtype, void* y, int ldy, int dtype, int rows, int n, int act,
+                                 float scale, cudaStream_t stream) {
+    TB_REQUIRE(x && g && y && rows > 0 && n > 0 && rows <= 65535 * 32, "gate_rows: rows are wanted (rows=%d n=%d)", rows, n);
+    TB_REQUIRE(act == 0 || act == 1, "gate_rows: the gate is a sigmoid (0) or silu (1)");
+    if (dtype == TB_F32 && g_dtype == TB_F32) launch_gate_rows<float, float>(x, ldx, g, ldg, y, ldy, rows, n, act, scale, stream);
+    else if (dtype == TB_BF16 && g_dtype == TB_BF16) launch_gate_rows<__nv_bfloat16, __nv_bfloat16>(x, ldx, g, ldg, y, ldy, rows, n, act, scale, stream);
+    else if (dtype == TB_BF16 && g_dtype == TB_F32) launch_gate_rows<__nv_bfloat16, float>(x, ldx, g, ldg, y, ldy, rows, n, act, scale, stream);
+    else TB_REQUIRE(false, "gate_rows: unsupported dtypes (rows %d, gate %d)", dtype, g_dtype);
     TB_CHECK_LAUNCH("gate_rows");
     return 0;
+}
+
+extern "C" int tb_gate_rows(const void* x, int ldx, const void* g, int ldg, void* y, int ldy, int dtype, int rows, int n, int act, float scale,
+                            cudaStream_t stream) {
+    return tb_gate_rows_from(x, ldx, g, ldg, dtype, y, ldy, dtype, rows, n, act, scale, stream);
 }
 
 extern "C" int tb_head_norm_gate_from(const float* o, int ldo, const float* w, int w_head, const void* g, int ldg, int g_dtype, void* y, int ldy,

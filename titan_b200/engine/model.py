@@ -35,8 +35,11 @@ class DecoderModel:
         return declare_weights(self.spec)
 
     def cache_needs(self) -> List[Optional[CacheNeed]]:
-        """One entry per RUN of the order, so a layer that runs twice keeps two caches."""
-        return [self.blocks[i].mixer.cache_need() for i in self.spec.order]
+        """One entry per RUN of the order, so a layer that runs twice keeps two caches: what the mixers need, and, where a
+        block keeps state of its own (``Block.own_need``), as many entries again for the blocks."""
+        mixers = [self.blocks[i].mixer.cache_need() for i in self.spec.order]
+        own = [b.own_need() if hasattr(b, "own_need") else None for b in (self.blocks[i] for i in self.spec.order)]
+        return mixers + own if any(n is not None for n in own) else mixers
 
     def cache_run_of(self, run: int) -> int:
         """The run whose cache the ``run``-th block of the order uses."""
@@ -89,6 +92,8 @@ class DecoderModel:
             x = x.repeat(1, streams)
         if "row_sums" not in ctx.scratch:      # places where folded norms leave sums of squares: one per run of a layer
             ctx.scratch["row_sums"] = torch.zeros((len(self.spec.order), 16, 32), dtype=torch.float32, device=ctx.device)
+        ctx.runs = len(self.spec.order)
+        ctx.block_state = lambda run: cache.view_for_layer(ctx.runs + run)
         for run, i in enumerate(self.spec.order):
             ctx.run = run
             ctx.next_block = self.blocks[self.spec.order[run + 1]] if run + 1 < len(self.spec.order) else None

@@ -90,7 +90,9 @@ class AttnArgs(Structure):
                 ("early_len", c_void_p), ("early_mode", c_int), ("fused_qk", POINTER(QkArgs)),
                 ("hd_v", c_int), ("v_alias", c_int), ("head_blocks", c_int), ("sink", c_void_p), ("keep_first", c_int),
                 ("softcap", c_float), ("rel_bias", c_void_p), ("rel_far", c_int), ("head_mix", c_void_p),
-                ("head_gate", c_void_p), ("head_gate_stride", c_int)]
+                ("head_gate", c_void_p), ("head_gate_stride", c_int),
+                ("pair_lambda", c_void_p), ("pair_eps", c_float), ("pair_scale", c_float), ("pair_width", c_int),
+                ("out_f32", c_int), ("exact_weights", c_int)]
 
 
 class LatentArgs(Structure):
@@ -107,7 +109,8 @@ class SplitAttnArgs(Structure):
     """Arguments of the tensor-core prompt attention with keys in two parts (csrc/attention_mma.cu: tb_attn_prefill_split)."""
     _fields_ = [("q", c_void_p), ("q_stride", c_int), ("kv", c_void_p), ("kv_stride", c_int), ("k_col0", c_int), ("v_col0", c_int),
                 ("tail", c_void_p), ("tail_stride", c_int), ("tail_col0", c_int), ("out", c_void_p), ("out_stride", c_int),
-                ("batch", Batch), ("nh", c_int), ("dn", c_int), ("dt", c_int), ("dv", c_int), ("window", c_int), ("scale", c_float)]
+                ("batch", Batch), ("nh", c_int), ("dn", c_int), ("dt", c_int), ("dv", c_int), ("window", c_int), ("scale", c_float),
+                ("sink", c_void_p), ("exact_weights", c_int)]
 
 
 class LightningArgs(Structure):
@@ -126,6 +129,30 @@ class WholeNormArgs(Structure):
                 ("pos_of", c_void_p), ("seq_of", c_void_p), ("slot_of_seq", c_void_p), ("kv_len", c_void_p),
                 ("cache", KvView), ("append", c_int), ("T", c_int),
                 ("o_bias", c_void_p), ("o_out", c_void_p), ("o_stride", c_int), ("o_width", c_int)]
+
+
+class PairPrepArgs(Structure):
+    """Arguments of the kernel between the projections of differential attention and its scores (csrc/differential.cu)."""
+    _fields_ = [("inp", c_void_p), ("in_stride", c_int), ("bias", c_void_p), ("q_w", c_void_p), ("k_w", c_void_p), ("eps", c_float),
+                ("q_out", c_void_p), ("q_stride", c_int), ("kv_out", c_void_p), ("kv_stride", c_int),
+                ("H", c_int), ("G", c_int), ("dim", c_int), ("vdim", c_int), ("hd", c_int),
+                ("pos_of", c_void_p), ("seq_of", c_void_p), ("slot_of_seq", c_void_p),
+                ("cache", KvView), ("append", c_int), ("T", c_int)]
+
+
+class SandwichArgs(Structure):
+    """Arguments of the kernel that adds a sublayer's normed output to the residual stream, with what may ride along (csrc/sandwich.cu)."""
+    _fields_ = [("y", c_void_p), ("post_w", c_void_p), ("post_eps", c_float), ("x", c_void_p), ("W", c_int), ("rows", c_int),
+                ("keep", c_void_p), ("hist", c_void_p), ("hist_stride", c_longlong), ("n_hist", c_int), ("dwa", c_void_p), ("store_hist", c_int),
+                ("pre_w", c_void_p), ("pre_eps", c_float), ("h", c_void_p),
+                ("mu", c_void_p), ("state", c_void_p), ("state_stride", c_longlong), ("slot_of_row", c_void_p)]
+
+
+class ShiftNormArgs(Structure):
+    """Arguments of the RMS norm with a token shift behind it (csrc/sandwich.cu)."""
+    _fields_ = [("x", c_void_p), ("W", c_int), ("rows", c_int), ("w", c_void_p), ("eps", c_float), ("mu", c_void_p), ("h", c_void_p),
+                ("state", c_void_p), ("state_stride", c_longlong), ("seq_of", c_void_p), ("q_start", c_void_p), ("slot_of_seq", c_void_p),
+                ("rows_per_block", c_int)]
 
 
 class WkvArgs(Structure):
@@ -204,6 +231,11 @@ def lib():
         l.tb_moe_route_scored.argtypes = [c_void_p, c_int, c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         l.tb_group_rmsnorm.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_float, c_void_p]
         l.tb_residual_group_norm.argtypes = [c_void_p, c_float, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]
+        l.tb_pair_prep.argtypes = [POINTER(PairPrepArgs), c_int, c_void_p]
+        l.tb_pair_combine.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p]
+        l.tb_sandwich_join.argtypes = [POINTER(SandwichArgs), c_int, c_void_p]
+        l.tb_shift_norm.argtypes = [POINTER(ShiftNormArgs), c_int, c_void_p]
+        l.tb_gate_rows_from.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_int, c_float, c_void_p]
         l.tb_qkv_whole_norm.argtypes = [POINTER(WholeNormArgs), c_int, c_void_p]
         l.tb_attn_mixed_prefill.argtypes = [POINTER(AttnArgs), c_int, c_void_p]
         l.tb_attn_mixed_decode.argtypes = [POINTER(AttnArgs), c_int, c_void_p]
@@ -456,12 +488,13 @@ GATE_SIGMOID, GATE_SILU = 0, 1
 
 
 def gate_rows(x: torch.Tensor, g: torch.Tensor, y: torch.Tensor, act: int, scale: float, stream: int) -> None:
-    """y = x * act(g) * scale, element by element (act GATE_SIGMOID or GATE_SILU, in float32); row-strided views of one dtype; y may be x."""
+    """y = x * act(g) * scale, element by element (act GATE_SIGMOID or GATE_SILU, in float32); row-strided views, x and y of one dtype, g in it
+    or in float32; y may be x."""
     _need_cuda(x, g, y)
-    if len({x.dtype, g.dtype, y.dtype}) != 1 or x.shape != g.shape or x.shape != y.shape or x.stride(1) != 1 or g.stride(1) != 1 or y.stride(1) != 1:
-        raise KernelError("gate_rows: three views of one dtype and shape are wanted")
-    _check(lib().tb_gate_rows(x.data_ptr(), x.stride(0), g.data_ptr(), g.stride(0), y.data_ptr(), y.stride(0), dtype_code(x.dtype), x.shape[0], x.shape[1],
-                              int(act), float(scale), stream))
+    if x.dtype != y.dtype or g.dtype not in (y.dtype, torch.float32) or x.shape != g.shape or x.shape != y.shape or x.stride(1) != 1 or g.stride(1) != 1 or y.stride(1) != 1:
+        raise KernelError("gate_rows: three views of one shape are wanted, the gate's in the rows' dtype or in float32")
+    _check(lib().tb_gate_rows_from(x.data_ptr(), x.stride(0), g.data_ptr(), g.stride(0), dtype_code(g.dtype), y.data_ptr(), y.stride(0),
+                                   dtype_code(x.dtype), x.shape[0], x.shape[1], int(act), float(scale), stream))
 
 
 def head_norm_gate(o: torch.Tensor, w: torch.Tensor, per_head: bool, g: torch.Tensor, y: torch.Tensor, heads: int, act: int, scale: float,
@@ -534,6 +567,60 @@ def residual_group_norm(y: torch.Tensor, mult: float, x: torch.Tensor, stream: i
         raise KernelError("residual_group_norm: contiguous float32 rows of one shape are wanted")
     _check(lib().tb_residual_group_norm(y.data_ptr(), float(mult), x.data_ptr(), _ptr(norm_w), _ptr(h),
                                         dtype_code(h.dtype) if h is not None else F32, x.shape[0], x.shape[1], groups, eps, stream))
+
+
+def pair_prep(args: "PairPrepArgs", dtype: torch.dtype, stream: int) -> None:
+    _check(lib().tb_pair_prep(byref(args), dtype_code(dtype), stream))
+
+
+def pair_combine(maps: torch.Tensor, hd: int, lam: torch.Tensor, out: torch.Tensor, width: int, eps: float, scale: float, stream: int) -> None:
+    """Per head h: o = maps[:, 2h] - lam * maps[:, 2h + 1] over its first ``width`` elements, over its root mean square, times
+    ``scale``.  maps float32 [T, 2 H hd], lam one float32 number on the device, out [T, H * width] in the compute dtype."""
+    _need_cuda(maps, lam, out)
+    H = out.shape[1] // width
+    if maps.dtype != torch.float32 or lam.dtype != torch.float32 or maps.stride(1) != 1 or out.stride(1) != 1 or out.shape[1] != H * width or maps.shape != (out.shape[0], 2 * H * hd):
+        raise KernelError("pair_combine: float32 rows of two maps a head and output rows of whole heads are wanted")
+    _check(lib().tb_pair_combine(maps.data_ptr(), maps.stride(0), hd, lam.data_ptr(), out.data_ptr(), out.stride(0), dtype_code(out.dtype), out.shape[0], H,
+                                 width, float(eps), float(scale), stream))
+
+
+def sandwich_join(y: torch.Tensor, post_w: torch.Tensor, post_eps: float, x: torch.Tensor, stream: int, keep: Optional[torch.Tensor] = None,
+                  history: Optional[torch.Tensor] = None, depth: int = 0, depth_w: Optional[torch.Tensor] = None,
+                  pre_w: Optional[torch.Tensor] = None, pre_eps: float = 0.0, h: Optional[torch.Tensor] = None,
+                  mu: Optional[torch.Tensor] = None, state: Optional[torch.Tensor] = None, slot_of_row: Optional[torch.Tensor] = None) -> None:
+    """x += rms(y) * post_w, y left zeroed (float32 rows).  ``keep`` receives x as it was.  ``history`` float32 [D, T, W] with ``depth`` rows
+    of it in place: the new row is put there as number ``depth`` (if D holds it) and x becomes sum_j depth_w[j] * row j, the new one
+    included.  ``h`` = rms(new x) * pre_w in h's dtype; with ``mu`` (every row a sequence's only token): h = g + (state[slot] - g) * mu
+    with g those normed rows, and state[slot] = g."""
+    _need_cuda(y, post_w, x, keep, history, depth_w, pre_w, h, mu, state, slot_of_row)
+    ok = lambda t: t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    if x.dtype != torch.float32 or y.shape != x.shape or not all(ok(t) for t in (y, post_w, x, keep, history, depth_w, pre_w, mu)) \
+            or (h is not None and (h.shape != x.shape or not h.is_contiguous())) or (state is not None and (state.dtype != torch.float32 or state.stride(1) != 1)) \
+            or (history is not None and (history.shape[1:] != x.shape or depth < 1 or depth > history.shape[0] or depth_w is None or depth_w.numel() != depth + 1)):
+        raise KernelError("sandwich_join: contiguous float32 rows of one shape, and a weight for every row of the history, are wanted")
+    a = SandwichArgs()
+    a.y, a.post_w, a.post_eps, a.x, a.W, a.rows = y.data_ptr(), post_w.data_ptr(), post_eps, x.data_ptr(), x.shape[1], x.shape[0]
+    a.keep = _ptr(keep)
+    if history is not None:
+        a.hist, a.hist_stride, a.n_hist, a.dwa = history.data_ptr(), history.stride(0), depth, depth_w.data_ptr()
+        a.store_hist = int(depth < history.shape[0])
+    a.pre_w, a.pre_eps, a.h = _ptr(pre_w), pre_eps, _ptr(h)
+    if mu is not None:
+        a.mu, a.state, a.state_stride, a.slot_of_row = mu.data_ptr(), state.data_ptr(), state.stride(0), slot_of_row.data_ptr()
+    _check(lib().tb_sandwich_join(byref(a), dtype_code(h.dtype) if h is not None else F32, stream))
+
+
+def shift_norm(x: torch.Tensor, w: torch.Tensor, eps: float, mu: torch.Tensor, h: torch.Tensor, state: torch.Tensor, layout, stream: int,
+               rows_per_block: int = 0) -> None:
+    """h = g + (g' - g) * mu with g = rms(x) * w (float32 rows in, h in its own dtype) and g' the previous token's g: the row before in the
+    same sequence, or the sequence's ``state`` row [slots, W] for its first row of the step; the state then holds its last row's g."""
+    _need_cuda(x, w, mu, h, state)
+    if any(t.dtype != torch.float32 or not t.is_contiguous() for t in (x, w, mu)) or h.shape != x.shape or not h.is_contiguous() \
+            or state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] != x.shape[1]:
+        raise KernelError("shift_norm: contiguous float32 rows and one state row per slot are wanted")
+    a = ShiftNormArgs(x.data_ptr(), x.shape[1], x.shape[0], w.data_ptr(), eps, mu.data_ptr(), h.data_ptr(), state.data_ptr(), state.stride(0),
+                      layout.seq_of.data_ptr(), layout.q_start.data_ptr(), layout.slot_of_seq.data_ptr(), int(rows_per_block))
+    _check(lib().tb_shift_norm(byref(a), dtype_code(h.dtype), stream))
 
 
 def qkv_whole_norm(args: "WholeNormArgs", out_dtype: torch.dtype, stream: int) -> None:

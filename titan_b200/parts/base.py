@@ -18,6 +18,8 @@ PositionEncoding  owned by a mixer; ``kernel_args(device)`` returns the argument
                 inverse frequencies, rotated dims, an offset on positions, a factor on cosines and
                 sines).  The default builds it from ``rotary_dim`` and ``tables(device)["inv_freq"]``.
 Block           ``forward(x_f32, ctx, cache)`` runs norms, mixer and feed-forward in its arrangement.
+                A block that keeps state of its own beside its mixer's says so in ``own_need() -> CacheNeed | None``
+                and finds it at ``ctx.block_state(run)``.
 
 All of them: ``weight_specs(prefix) -> [WeightSpec]`` and ``bind(get)``, where
 ``get(relative_name) -> tensor`` hands out the declared tensors on the device.

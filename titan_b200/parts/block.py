@@ -5,7 +5,7 @@ its first matrix product is handed over unevaluated (``norm.DeferredNorm``)
 (berniehans/titan: engine/engine-core/src/forward_cpu.rs:281-386).  The
 residual stream ``x`` is float32 and is updated in place: mixer and
 feed-forward add into it in the epilogue of their last matrix product.  The other arrangements (``pre_norm_scaled``,
-``output_norm``, ``hyper``, ``parallel``) are described at their classes.
+``output_norm``, ``hyper``, ``parallel``, ``sandwich``) are described at their classes.
 """
 from __future__ import annotations
 
@@ -13,6 +13,7 @@ from typing import List
 
 import torch
 
+from ..cache.groups import CacheNeed
 from ..weights.loader import WeightSpec
 from .base import BLOCKS, FEED_FORWARDS, MIXERS, NORMS, Part
 
@@ -374,3 +375,125 @@ class ParallelBlock(Part):
 
 
 BLOCKS.register("parallel", ParallelBlock)
+
+
+class SandwichBlock(Part):
+    """``sandwich``: a norm before AND after each sublayer, each if asked: a token shift in front of the mixer, and an average
+    over depth behind the block:
+
+        h = norm1(x);  h_t <- h_t + (h_{t-1} - h_t) * s;   x += norm1b(mixer(h));   x += norm2b(feed_forward(norm2(x)))
+        x <- sum over j = 0 .. i + 1 of w_j X_j             X_0 the rows that entered the first block, X_{j+1} what block j made
+
+    ``LayerSpec.norms`` are the norms after the sublayers (one a sublayer; the feed-forward, with both its norms, may be
+    absent).  ``LayerSpec.extra``: "token_shift" = name of the factors s [W]; "depth_average" = (name of the weights w [i + 2], i)
+    with i the block's place in the running order.
+
+    A sublayer adds into a zeroed float32 buffer of the step; ONE kernel then norms that buffer, adds it to the residual stream,
+    leaves it zeroed and goes on with what follows: the feed-forward's normed input, or the average over depth and, where
+    the next block is of this arrangement, the rows its mixer reads.  With a token shift those need the previous token's row:
+    in a step of single tokens that is the sequence's state, so the same kernel shifts too; in a step of longer runs the next
+    block's own kernel norms and shifts (the row before is a neighbour's).  The previous token's normed row, before its own
+    shift, is the block's state: float32, one row a sequence and run, in a ``state`` cache group (zero at a sequence's start).
+    The rows X_j live in a buffer of the step ([runs, T, W] float32): nothing of them outlasts it."""
+
+    def __init__(self, spec):
+        if spec.mixer_norm is None or (spec.feed_forward is None) != (spec.feed_forward_norm is None) or len(spec.norms) != (1 if spec.feed_forward is None else 2):
+            raise ValueError("the sandwich arrangement takes a norm before and a norm after the mixer, and a feed-forward with two norms of its own or none")
+        for n in (spec.mixer_norm, spec.feed_forward_norm) + tuple(spec.norms):
+            if n is not None and (n.kind != "rmsnorm" or getattr(n, "groups", 1) != 1):
+                raise ValueError("the sandwich arrangement folds plain RMS norms (one group) into the kernels around its sublayers")
+        self.spec = spec
+        self.W = spec.mixer.hidden_size
+        self.mixer_norm = NORMS.build(spec.mixer_norm)
+        self.mixer = MIXERS.build(spec.mixer)
+        self.feed_forward_norm = None if spec.feed_forward_norm is None else NORMS.build(spec.feed_forward_norm)
+        self.feed_forward = None if spec.feed_forward is None else FEED_FORWARDS.build(spec.feed_forward)
+        self.after = [NORMS.build(n) for n in spec.norms]
+        self.shift_name = spec.option("token_shift")
+        self.depth_name, self.place = spec.option("depth_average", (None, 0))
+        self.shift = self.depth_w = None
+
+    def parts(self):
+        ffn = () if self.feed_forward is None else (self.feed_forward_norm, self.feed_forward)
+        return (self.mixer_norm, self.mixer) + ffn + tuple(self.after)
+
+    def own_need(self):
+        return None if self.shift_name is None else CacheNeed("state", state_shape=(self.W,), state_dtype=torch.float32)
+
+    def weight_specs(self, prefix: str = "") -> List[WeightSpec]:
+        out: List[WeightSpec] = []
+        for part in self.parts():
+            out += part.weight_specs(self.spec.prefix)
+        if self.shift_name is not None:
+            out.append(WeightSpec(self.spec.prefix + self.shift_name, (self.W,), "vector", ("normal_around", 0.2, 0.3)))
+        if self.depth_name is not None:
+            n = self.place + 2
+            out.append(WeightSpec(self.spec.prefix + self.depth_name, (n,), "vector", ("normal_around", 0.2, 1.0 / n)))
+        return out
+
+    def bind(self, get) -> None:
+        for part in self.parts():
+            part.bind(lambda name: get(self.spec.prefix + name))
+        if self.shift_name is not None:
+            self.shift = get(self.spec.prefix + self.shift_name).contiguous()
+        if self.depth_name is not None:
+            self.depth_w = get(self.spec.prefix + self.depth_name).contiguous()
+
+    @staticmethod
+    def _state(ctx, run):
+        group, index = ctx.block_state(run)
+        return group.layer_storage(index)
+
+    def _read(self, x, ctx):
+        """The mixer's input rows, by kernels of their own."""
+        if self.shift is None:
+            return self.mixer_norm.forward(x, ctx)
+        from .. import kernels as K
+        h = ctx.empty(tuple(x.shape))
+        K.shift_norm(x, self.mixer_norm.weight, self.mixer_norm.spec.eps, self.shift, h, self._state(ctx, ctx.run), ctx.layout, ctx.stream)
+        return h
+
+    def _following(self, x, ctx):
+        """What the kernel at this block's end may make for the next block: keyword arguments of the join, the next mixer's rows among them."""
+        nxt = ctx.next_block
+        if not isinstance(nxt, SandwichBlock) or nxt.W != self.W or not ctx.options.get("fuse_sandwich", True):
+            return {}
+        if nxt.shift is not None and not ctx.layout.all_single:
+            return {}
+        made = dict(pre_w=nxt.mixer_norm.weight, pre_eps=nxt.mixer_norm.spec.eps, h=ctx.empty(tuple(x.shape)))
+        if nxt.shift is not None:
+            made.update(mu=nxt.shift, state=self._state(ctx, ctx.run + 1), slot_of_row=ctx.layout.slot_of_seq)
+        return made
+
+    def forward(self, x: torch.Tensor, ctx, cache) -> None:
+        from .. import kernels as K
+        y = ctx.carried.get("sublayer_sum")
+        if y is None or y.shape != x.shape:
+            y = ctx.carried["sublayer_sum"] = torch.zeros_like(x)         # zeroed once a step; the joining kernel leaves it zeroed
+        history = keep = None
+        if self.depth_w is not None:
+            if ctx.run != self.place:
+                raise RuntimeError(f"a block with {self.place + 2} depth weights runs as number {ctx.run}")
+            history = ctx.carried.get("depth_rows")
+            if ctx.run == 0:                                              # the rows that enter the first block are depth 0: its first join keeps them
+                history = ctx.carried["depth_rows"] = ctx.empty((ctx.runs,) + tuple(x.shape), torch.float32)
+                keep = history[0]
+            elif history is None:
+                raise RuntimeError("an average over depth needs every block from the first on to keep its rows")
+        kept = ctx.carried.pop("normed_rows", None)
+        h = kept[0] if kept is not None and kept[1] == ctx.run and kept[0].shape == x.shape else self._read(x, ctx)
+        self.mixer.forward(h, ctx, cache, y)
+        if self.feed_forward is not None:
+            n1, n2 = self.after[0], self.feed_forward_norm
+            h = ctx.empty(tuple(x.shape))
+            K.sandwich_join(y, n1.weight, n1.spec.eps, x, ctx.stream, keep=keep, pre_w=n2.weight, pre_eps=n2.spec.eps, h=h)
+            keep = None
+            self.feed_forward.forward(h, ctx, y)
+        made, n = self._following(x, ctx), self.after[-1]
+        K.sandwich_join(y, n.weight, n.spec.eps, x, ctx.stream, keep=keep, history=history, depth=self.place + 1 if history is not None else 0,
+                        depth_w=self.depth_w, **made)
+        if made:
+            ctx.carried["normed_rows"] = (made["h"], ctx.run + 1)
+
+
+BLOCKS.register("sandwich", SandwichBlock)

@@ -18,6 +18,11 @@ NormSpec), q = c_q . W_uq^T (tensor roles "dq" and "uq" instead of "q"); the pro
 k_raw] as two products (query latent; latent and key part), a norm kernel makes c_q, and a third product fills the query
 columns of the row that the prep kernel reads.
 
+With the option ``sink`` (the name of a tensor with one number a head) a head's softmax denominator also contains exp(sink), once,
+without a key.  With ``out_gate`` (the name of a [heads * value_dim, hidden] tensor) the concatenated heads are multiplied by
+sigmoid(W_g h) before the output projection; the gate's logits are further columns of the float32 input product.  With
+``exact_weights`` the tensor-core prompt kernel multiplies the values by the softmax weights as two bfloat16 halves.
+
 Rows are padded with zeros to a multiple of 8 elements.  A mixer with ``cache_from`` has no W_dkv: it reads the rows
 of the named layer (its own window may be shorter than what that layer keeps).  A step of single tokens appends in
 the prep kernel and attends over the cache; a step with longer runs attends over cache + the step's own rows (the
@@ -66,6 +71,8 @@ class LatentAttentionMixer(Mixer):
         if self.q_rank and self.q_norm_spec is None:
             raise ValueError("queries through a latent need that latent's norm (q_norm)")
         self.w_uq = self.q_norm = self.w_dkv = None
+        self.sink_name, self.gate_name, self.exact = s.option("sink"), s.option("out_gate"), bool(s.option("exact_weights", False))
+        self.sink = self.w_gate = None
         self.scale = s.softmax_scale if s.softmax_scale is not None else 1.0 / math.sqrt(self.dn + self.rd)
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.latent_w = None
         self._views = {}
@@ -91,6 +98,10 @@ class LatentAttentionMixer(Mixer):
         if not self.shared:
             specs.append(WeightSpec(p + n["dkv"], (self.r + self.rd, W)))
             specs += NORMS.build(self.latent_norm_spec).weight_specs(p)
+        if self.sink_name:
+            specs.append(WeightSpec(p + self.sink_name, (self.H,), "vector", ("normal", 1.0)))
+        if self.gate_name:
+            specs.append(WeightSpec(p + self.gate_name, (self.H * self.dv, W)))
         specs += [WeightSpec(p + n["uk"], (self.H * self.dn, self.r)), WeightSpec(p + n["uv"], (self.H * self.dv, self.r)),
                   WeightSpec(p + n["o"], (W, self.H * self.dv))]
         return specs
@@ -113,6 +124,16 @@ class LatentAttentionMixer(Mixer):
             norm = NORMS.build(self.latent_norm_spec)
             norm.bind(lambda name: get(p + name))
             self.latent_w = norm.weight
+        if self.sink_name:
+            self.sink = get(p + self.sink_name).contiguous()
+        if self.gate_name:
+            if self.q_rank:                                    # the input product is of another kind: the gate is a product of its own
+                self.w_gate = get(p + self.gate_name)
+            else:                                              # the gate's logits behind the other columns, on a 16-byte border
+                g = get(p + self.gate_name)
+                pad = -self.w_in.shape[0] % 8
+                self.gate_col = self.w_in.shape[0] + pad
+                self.w_in = torch.cat([self.w_in] + ([g.new_zeros((pad, g.shape[1]))] if pad else []) + [g], dim=0).contiguous()
         # U_k by head, transposed: [H, kv_rank, dim], so that q~_h = q_h . (that)^T; U_v by head as stored: [H, vdim, kv_rank]
         uk, uv = get(p + n["uk"]), get(p + n["uv"])
         self.w_uk_t = uk.view(self.H, self.dn, self.r).transpose(1, 2).contiguous()
@@ -148,6 +169,8 @@ class LatentAttentionMixer(Mixer):
         a.batch = lay.c_struct()
         a.nh, a.dn, a.dt, a.dv = self.H, self.dn, self.rd, self.dv
         a.window, a.scale = s.window or 0, self.scale
+        a.sink = None if self.sink is None else self.sink.data_ptr()
+        a.exact_weights = int(self.exact and bool(ctx.options.get("exact_weights", True)))
         return a if K.attn_prefill_split_accepts(a) else None
 
     def forward(self, h, ctx, cache, out: torch.Tensor) -> None:
@@ -212,6 +235,7 @@ class LatentAttentionMixer(Mixer):
             linear.matmul(rows[:, :r], self.w_ukv, kv, linear.EPI_STORE, ctx)
             o = ctx.empty((T, H * dv))
             K.attn_prefill_split(self._split_args(ctx, q_full, kv, rows, o), ctx.stream)
+            self._gate(o, h, proj, ctx)
             linear.matmul(o, self.w_o, out, linear.EPI_ADD, ctx)
             return
         # the heads' unrotated queries into the latent space
@@ -224,6 +248,7 @@ class LatentAttentionMixer(Mixer):
         aa.cache, aa.batch = view, lay.c_struct()
         aa.nh, aa.nkv, aa.hd, aa.hd_v, aa.v_alias = H, 1, dk, r, 1
         aa.window, aa.scale = s.window or 0, self.scale
+        aa.sink = None if self.sink is None else self.sink.data_ptr()
         if decode:
             # all heads read one row per key: a block for every few heads (not one for the single "kv head"), and splits
             # of one page, or of half a page while that still leaves SMs without a block (a step of one or two sequences:
@@ -246,7 +271,19 @@ class LatentAttentionMixer(Mixer):
         # out of the latent space, head by head, and through the output projection
         o = ctx.empty((T, H * dv))
         linear.matmul_heads(lat, self.w_uv, o, H, r, dv, ctx)
+        self._gate(o, h, proj, ctx)
         linear.matmul(o, self.w_o, out, linear.EPI_ADD, ctx)
+
+    def _gate(self, o: torch.Tensor, h, proj: torch.Tensor, ctx) -> None:
+        """The concatenated heads times sigmoid(W_g h), in place, where the layer has such a gate."""
+        if not self.gate_name:
+            return
+        if self.w_gate is not None:
+            logits = ctx.empty((o.shape[0], self.H * self.dv), torch.float32)
+            linear.matmul(h, self.w_gate, logits, linear.EPI_F32, ctx)
+        else:
+            logits = proj[:, self.gate_col:self.gate_col + self.H * self.dv]
+        K.gate_rows(o, logits, o, K.GATE_SIGMOID, 1.0, ctx.stream)
 
 
 MIXERS.register("latent_attention", LatentAttentionMixer)
