@@ -640,6 +640,20 @@ def desalorn_config(width, layers, heads, experts, top, ff, shared_ff, window, v
             "embedding": {"scale": 1.0}, "layers": out}
 
 
+def pipesun_config(width, layers, heads, experts, top, ff, shared_ff, window, vocab=32768):
+    """A Pipesun model of the same sizes (without windows and mixtures, which the design does not have): latent attention (heads of
+    128 + 64, a latent of 512) with a sink and a gate, differential attention (two maps of 64 a head, values of 128, a quarter as many
+    kv heads), latent attention, differential attention on the earlier one's keys and values; dense feed-forwards as wide as what a
+    token uses of a mixture."""
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "rot": {"base": 10000.0, "dims": 64}, "scale": 1.0 / (192 ** 0.5)}
+    diff = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.4}
+    out = []
+    for i in range(layers):
+        m = latent if i % 2 == 0 else (diff if i % 4 == 1 else dict(diff, kv_from=i - 2))
+        out.append({"type": "latent_attention" if i % 2 == 0 else "attention", "mixer": dict(m), "mlp": {"kind": "dense", "ff": top * ff + shared_ff}})
+    return {"architecture": "Pipesun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
+
+
 def qwen3_like(width, layers, heads, ffn, vocab=32768):
     """The dense model of equal size: the same width, depth and heads, and a feed-forward as wide as what one token uses
     of the mixture (its chosen experts and the shared one)."""
@@ -657,7 +671,7 @@ def launcher_times(engine, torch, K, entries):
                          "gated_rmsnorm", "moe_route", "token_gate_rows", "moe_plan", "moe_grouped", "moe_rows", "moe_combine", "moe_experts_tc",
                          "dyt", "scale_add", "wkv", "moe_route_all", "hyper", "polynorm", "gate_rows", "head_norm_gate", "delta_prep",
                          "recurrent_scan", "group_rmsnorm", "residual_group_norm", "qkv_whole_norm", "attn_mixed_prefill", "attn_mixed_decode",
-                         "rotary_rows", "moe_route_scored") if hasattr(K, n)]
+                         "rotary_rows", "moe_route_scored", "pair_prep", "pair_combine", "sandwich_join", "shift_norm") if hasattr(K, n)]
     events, originals = [], {n: getattr(K, n) for n in names}
 
     def wrap(name, f):
@@ -688,11 +702,12 @@ def launcher_times(engine, torch, K, entries):
 
 
 def run_design(args):
-    """``--design tefezen | zadinex | vuvosun | desalorn``: prompt and decode throughput of that design at sizes that resemble a
+    """``--design tefezen | zadinex | vuvosun | desalorn | pipesun``: prompt and decode throughput of that design at sizes that resemble a
     served model's layers (random weights), beside the Qwen3 dense model of equal size and beside the closest design (for zadinex:
     Tefezen, windowed attention, a recurrence, mixtures of experts; for vuvosun: Zadinex with dense feed-forwards, attention
     with a sink and a recurrence over a matrix state; for desalorn: Tefezen, latent attention over a window, decayed linear
-    attention, mixtures of experts with a shared one), and where a step's time goes by launcher."""
+    attention, mixtures of experts with a shared one; for pipesun: Tefezen too, for its latent attention and the norms on its
+    sublayers' outputs), and where a step's time goes by launcher."""
     import torch
 
     from titan_b200 import Engine, StepEntry, kernels as K
@@ -707,9 +722,11 @@ def run_design(args):
     for sz in sizes:
         row = {"size": sz}
         beside = {"tefezen": ("qwen3",), "zadinex": ("tefezen", "qwen3"), "vuvosun": ("zadinex_dense", "qwen3"),
-                  "desalorn": ("tefezen", "qwen3")}[args.design]
+                  "desalorn": ("tefezen", "qwen3"), "pipesun": ("tefezen", "qwen3")}[args.design]
         for which in (args.design,) + beside:
-            if which == "desalorn":
+            if which == "pipesun":
+                cfg = pipesun_config(**sz)
+            elif which == "desalorn":
                 cfg = desalorn_config(**sz)
             elif which == "vuvosun":
                 cfg = vuvosun_config(**sz)
@@ -766,7 +783,7 @@ def main():
     ap.add_argument("--micro", action="store_true", help="time the layer's kernels alone (CUDA events) and exit; text lines, not the JSON line")
     ap.add_argument("--timeline", type=int, default=0, metavar="BATCH", help="when the CTAs of one captured decode step's kernels start, wait and end "
                     "(needs TITAN_B200_NVCC_FLAGS=-DTB_TIMELINE); text lines, not the JSON line")
-    ap.add_argument("--design", default=None, choices=["tefezen", "zadinex", "vuvosun", "desalorn"], help="prompt and decode throughput of another design at a few sizes beside "
+    ap.add_argument("--design", default=None, choices=["tefezen", "zadinex", "vuvosun", "desalorn", "pipesun"], help="prompt and decode throughput of another design at a few sizes beside "
                     "the dense model of equal size; one JSON line of its own, the default workload is not run")
     ap.add_argument("--design-size", type=int, default=None, choices=[0, 1], help="with --design: one of its sizes only")
     args = ap.parse_args()
