@@ -228,62 +228,92 @@ __global__ void __launch_bounds__(ATT_WARPS * 32) attn_decode_kernel(AttnArgs a)
     }
 }
 
-// The splits of one head in order: acc = sum_s exp(m_s - m) acc_s, returned unnormalised, with l = sum_s exp(m_s - m) l_s
-// (the sink's term included).  Every thread finds the maximum and the weights' sum itself from the splits' (m, l) pairs (a
-// few broadcast loads) and adds up its own output dims, so the loads of different splits do not wait for one another; splits
-// that saw no key (all of them before a window's first key) are skipped.
-template <int PER>
-__device__ __forceinline__ float merge_splits(const AttnArgs& a, int b, int h, int hd, int used, int first, float* acc) {
-    const int stride = hd + 2;
-    const float* part = a.scratch + (size_t)(b * a.nh + h) * a.n_splits * stride;
-    float m = -FLT_MAX;
-    for (int s = first; s < used; ++s)
-        if (part[s * stride + hd + 1] > 0.f) m = fmaxf(m, part[s * stride + hd]);
-    const bool sunk = a.sink != nullptr;
-    if (sunk) m = fmaxf(m, a.sink[h]);
-    float l = 0.f;
+// The splits of NH neighbouring heads (h0 ..) merged for output dims ``d0 + threadIdx.x + blockDim.x * j``: acc[k][j] =
+// sum_s exp(m_s - m) acc_s and l[k] = sum_s exp(m_s - m) l_s (the sink's term included), both in the order of the splits.  The
+// block first turns the splits' (m, l) pairs into weights, a thread a split, MERGE_TILE splits at a time; the loads of the
+// sums then wait for nothing but the weights in shared memory.  Splits that saw no key (l = 0) get the weight zero.
+#define MERGE_TILE 128
+template <int NH, int PER>
+__device__ __forceinline__ void merge_splits(const AttnArgs& a, int b, int h0, int hd, int d0, int used, int first, float (&acc)[NH][PER], float (&l)[NH]) {
+    __shared__ float sm[NH][MERGE_TILE], sl[NH][MERGE_TILE], red[NH][32];
+    const int stride = hd + 2, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
+    const float* part = a.scratch + (size_t)(b * a.nh + h0) * a.n_splits * stride;
+    const size_t head = (size_t)a.n_splits * stride;
+    float m[NH];
 #pragma unroll
-    for (int j = 0; j < PER; ++j) acc[j] = 0.f;
-    for (int s = first; s < used; ++s) {
-        const float ls = part[s * stride + hd + 1];
-        if (!(ls > 0.f)) continue;
-        const float w = expf(part[s * stride + hd] - m);
-        l = fmaf(w, ls, l);
-        const float* p = part + (size_t)s * stride;
+    for (int k = 0; k < NH; ++k) {
+        m[k] = -FLT_MAX; l[k] = 0.f;
 #pragma unroll
-        for (int j = 0; j < PER; ++j) {
-            const int d = threadIdx.x + blockDim.x * j;
-            if (d < hd) acc[j] = fmaf(w, p[d], acc[j]);
-        }
+        for (int j = 0; j < PER; ++j) acc[k][j] = 0.f;
     }
-    if (sunk) l += expf(a.sink[h] - m);               // the sink counts once, here, not once a split
-    return l;
+    // the first tile's pairs stay in shared memory; the maximum runs over all of them
+    for (int s = threadIdx.x; s < used - first; s += blockDim.x)
+#pragma unroll
+        for (int k = 0; k < NH; ++k) {
+            const float* p = part + k * head + (size_t)(first + s) * stride + hd;
+            const float ms = p[0], ls = p[1];
+            if (ls > 0.f) m[k] = fmaxf(m[k], ms);
+            if (s < MERGE_TILE) { sm[k][s] = ms; sl[k][s] = ls; }
+        }
+#pragma unroll
+    for (int k = 0; k < NH; ++k) {
+        m[k] = warp_max(m[k]);
+        if (lane == 0) red[k][warp] = m[k];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < NH; ++k) {
+        for (int w = 0; w < nwarp; ++w) m[k] = fmaxf(m[k], red[k][w]);
+        if (a.sink) m[k] = fmaxf(m[k], a.sink[h0 + k]);
+    }
+    for (int s0 = 0; s0 < used - first; s0 += MERGE_TILE) {
+        const int n = min(MERGE_TILE, used - first - s0);
+        if (s0 > 0) __syncthreads();
+        for (int s = threadIdx.x; s < n; s += blockDim.x)
+#pragma unroll
+            for (int k = 0; k < NH; ++k) {
+                const float* p = part + k * head + (size_t)(first + s0 + s) * stride + hd;
+                const float ms = s0 > 0 ? p[0] : sm[k][s], ls = s0 > 0 ? p[1] : sl[k][s];      // (a thread reads back what it wrote itself)
+                const float w = ls > 0.f ? expf(ms - m[k]) : 0.f;
+                sm[k][s] = w; sl[k][s] = w * ls;
+            }
+        __syncthreads();
+        const float* p = part + (size_t)(first + s0) * stride + d0 + threadIdx.x;
+#pragma unroll 8
+        for (int s = 0; s < n; ++s)
+#pragma unroll
+            for (int k = 0; k < NH; ++k) {
+                const float w = sm[k][s];
+                l[k] += sl[k][s];
+#pragma unroll
+                for (int j = 0; j < PER; ++j)
+                    if (d0 + (int)threadIdx.x + (int)blockDim.x * j < hd) acc[k][j] = fmaf(w, p[k * head + (size_t)s * stride + blockDim.x * j], acc[k][j]);
+            }
+    }
+    if (a.sink)                                        // the sink counts once, here, not once a split
+#pragma unroll
+        for (int k = 0; k < NH; ++k) l[k] += expf(a.sink[h0 + k] - m[k]);
 }
 
-// grid (B, nh), one block of up to 128 threads: out = sum_s exp(m_s - m) acc_s / sum_s exp(m_s - m) l_s.
-template <typename T, int MAXE>
-__global__ void attn_merge_kernel(AttnArgs a) {
+// grid (B, nh, ceil(value width / 128)), 128 threads: out = sum_s exp(m_s - m) acc_s / sum_s exp(m_s - m) l_s.
+template <typename T>
+__global__ void __launch_bounds__(128) attn_merge_kernel(AttnArgs a) {
     pdl_launch_dependents();
     pdl_wait();
-    const int b = blockIdx.x, h = blockIdx.y, hd = value_width(a);
+    const int b = blockIdx.x, h = blockIdx.y, hd = value_width(a), d = blockIdx.z * 128 + threadIdx.x;
     const int len = a.batch.kv_len[b], keys = tb_split_keys(len, a.chunk, a.n_splits);
     const int used = min(a.n_splits, (len + keys - 1) / keys);
     const int first = (a.window > 0 && a.keep_first <= 0) ? max(0, len - a.window) / keys : 0;      // splits before the window's first key hold nothing
-    constexpr int PER = (32 * MAXE + 127) / 128;
-    float acc[PER];
-    float inv = 1.0f / merge_splits<PER>(a, b, h, hd, used, first, acc);
+    float acc[1][1], l[1];
+    merge_splits<1, 1>(a, b, h, hd, blockIdx.z * 128, used, first, acc, l);
+    float inv = 1.0f / l[0];
     if (a.head_gate) inv *= 1.0f / (1.0f + expf(-a.head_gate[(size_t)b * a.head_gate_stride + h]));      // the head's gate
-    T* o = (T*)a.out + (size_t)b * a.out_stride + h * hd;
-#pragma unroll
-    for (int j = 0; j < PER; ++j) {
-        const int d = threadIdx.x + blockDim.x * j;
-        if (d < hd) stf(o + d, acc[j] * inv);
-    }
+    if (d < hd) stf((T*)a.out + (size_t)b * a.out_stride + h * hd + d, acc[0][0] * inv);
 }
 
 // grid (B, nh / 2), 128 threads: both maps of a pair merged, the second times lambda taken off the first, the difference
 // divided by its root mean square (AttnArgs.pair_lambda).
-template <typename T, int MAXE>
+template <typename T, int PER>
 __global__ void __launch_bounds__(128) attn_merge_pair_kernel(AttnArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -292,24 +322,22 @@ __global__ void __launch_bounds__(128) attn_merge_pair_kernel(AttnArgs a) {
     const int len = a.batch.kv_len[b], keys = tb_split_keys(len, a.chunk, a.n_splits);
     const int used = min(a.n_splits, (len + keys - 1) / keys);
     const int first = (a.window > 0 && a.keep_first <= 0) ? max(0, len - a.window) / keys : 0;
-    constexpr int PER = (32 * MAXE + 127) / 128;
-    float a1[PER], a2[PER];
-    const float inv1 = 1.0f / merge_splits<PER>(a, b, 2 * p, hd, used, first, a1);
-    const float inv2 = 1.0f / merge_splits<PER>(a, b, 2 * p + 1, hd, used, first, a2);
-    const float lam = *a.pair_lambda;
+    float acc[2][PER], l[2];
+    merge_splits<2, PER>(a, b, 2 * p, hd, 0, used, first, acc, l);
+    const float lam = *a.pair_lambda, inv1 = 1.0f / l[0], inv2 = 1.0f / l[1];
     float ss = 0.f;
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
-        const int d = threadIdx.x + blockDim.x * j;
-        a1[j] = d < a.pair_width ? fmaf(-lam, a2[j] * inv2, a1[j] * inv1) : 0.f;
-        ss = fmaf(a1[j], a1[j], ss);
+        const int d = threadIdx.x + 128 * j;
+        acc[0][j] = d < a.pair_width ? fmaf(-lam, acc[1][j] * inv2, acc[0][j] * inv1) : 0.f;
+        ss = fmaf(acc[0][j], acc[0][j], ss);
     }
     const float r = a.pair_scale / sqrtf(block_sum(ss, red) / (float)a.pair_width + a.pair_eps);
     T* o = (T*)a.out + (size_t)b * a.out_stride + p * a.pair_width;
 #pragma unroll
     for (int j = 0; j < PER; ++j) {
-        const int d = threadIdx.x + blockDim.x * j;
-        if (d < a.pair_width) stf(o + d, a1[j] * r);
+        const int d = threadIdx.x + 128 * j;
+        if (d < a.pair_width) stf(o + d, acc[0][j] * r);
     }
 }
 
@@ -361,12 +389,23 @@ extern "C" int tb_attn_prefill(const AttnArgs* args, int dtype, cudaStream_t str
 extern "C" int tb_attn_merge(const AttnArgs* args, int dtype, cudaStream_t stream) {
     AttnArgs a = *args;
     TB_REQUIRE(dtype == TB_F32 || dtype == TB_BF16, "attn_merge: unknown dtype %d", dtype);
-    const bool wide = wide_rows(a);
+    const int width = value_width(a);
     if (a.pair_lambda) {
-        TB_REQUIRE(a.nh % 2 == 0 && a.pair_width > 0 && a.pair_width <= value_width(a) && !a.head_gate && !a.sink, "attn_merge: pairs of heads do not fit");
-        ATT_DISPATCH(attn_merge_pair_kernel, dim3(a.batch.B, a.nh / 2), 128, 0);
+        TB_REQUIRE(a.nh % 2 == 0 && a.pair_width > 0 && a.pair_width <= width && !a.head_gate && !a.sink, "attn_merge: pairs of heads do not fit");
+        const dim3 grid(a.batch.B, a.nh / 2);
+        if (dtype == TB_F32) {
+            if (width <= 128) tb_launch(attn_merge_pair_kernel<float, 1>, grid, 128, 0, stream, a);
+            else if (width <= 256) tb_launch(attn_merge_pair_kernel<float, 2>, grid, 128, 0, stream, a);
+            else tb_launch(attn_merge_pair_kernel<float, 8>, grid, 128, 0, stream, a);
+        } else {
+            if (width <= 128) tb_launch(attn_merge_pair_kernel<__nv_bfloat16, 1>, grid, 128, 0, stream, a);
+            else if (width <= 256) tb_launch(attn_merge_pair_kernel<__nv_bfloat16, 2>, grid, 128, 0, stream, a);
+            else tb_launch(attn_merge_pair_kernel<__nv_bfloat16, 8>, grid, 128, 0, stream, a);
+        }
     } else {
-        ATT_DISPATCH(attn_merge_kernel, dim3(a.batch.B, a.nh), 128, 0);
+        const dim3 grid(a.batch.B, a.nh, (width + 127) / 128);
+        if (dtype == TB_F32) tb_launch(attn_merge_kernel<float>, grid, 128, 0, stream, a);
+        else tb_launch(attn_merge_kernel<__nv_bfloat16>, grid, 128, 0, stream, a);
     }
     TB_CHECK_LAUNCH("attn_merge");
     return 0;

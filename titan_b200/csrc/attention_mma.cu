@@ -20,12 +20,14 @@
 
 #include "attention_args.h"
 #include "common.cuh"
+#include "mma.cuh"
 #include "timeline.cuh"
 #include "tma.cuh"
 
 namespace {
 
 using namespace tbtma;
+using namespace tbmma;
 
 __device__ unsigned int g_attn_error = 0;
 
@@ -60,29 +62,6 @@ struct DecArgs {
     const float* sink;                             // [nh] or null: one more term exp(sink) of every head's softmax denominator
     int keep_first;                                // with a window: the sequence's first keep_first keys stay visible
 };
-
-__device__ __forceinline__ void ldsm_x4(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t& r0, uint32_t& r1, uint32_t& r2, uint32_t& r3) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float* c, uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack2(float lo, float hi) {
-    const __nv_bfloat162 p = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&p);
-}
-// The two parts of (lo, hi) that rounding them to the pair ``rounded`` left over, themselves rounded.
-__device__ __forceinline__ uint32_t rest2(float lo, float hi, uint32_t rounded) {
-    return pack2(lo - __uint_as_float(rounded << 16), hi - __uint_as_float(rounded & 0xffff0000u));
-}
-// Byte offset of (row, 16-byte chunk of the row's 128 bytes) in a 64-row, 128-byte-swizzled box.
-__device__ __forceinline__ uint32_t swz(int row, int chunk16) { return (uint32_t)(row * 128 + ((chunk16 ^ (row & 7)) << 4)); }
 
 // HD: head size (64 or 128).  WIDE: the group has more than 8 query heads (rows 8..15 of the tile are live).
 // CL: the splits of a (sequence, kv head) are the CTAs of one thread-block cluster (up to 16).  Every CTA merges a

@@ -34,7 +34,7 @@ from typing import List, Optional
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 LIBS = {"core": "libtitan_b200.so", "tensor": "libtitan_b200_tensor.so", "attention": "libtitan_b200_attention.so"}
-SOURCES_OF = {"tensor": ("gemm_tc.cu", "tma_host.cu"), "attention": ("attention_mma.cu", "attention_tc.cu")}
+SOURCES_OF = {"tensor": ("gemm_tc.cu", "tma_host.cu"), "attention": ("attention_latent.cu", "attention_mma.cu", "attention_tc.cu")}
 LOADS_FIRST = {"core": None, "tensor": "core", "attention": "tensor"}
 ARCH_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a"]
 NVCC_FLAGS = ["-O3", "-std=c++17", "-lineinfo", "-Xcompiler", "-fPIC", "--expt-relaxed-constexpr",

@@ -48,7 +48,8 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a) {
     pdl_wait();
     extern __shared__ float sm[];
     __shared__ float red[33];
-    const int t = blockIdx.x;
+    // grid (T, parts): the blocks of a token take its heads in turns; the first one makes the cache row as well
+    const int t = blockIdx.x, h0 = blockIdx.y, h_step = gridDim.y;
     const int half = a.rope.rot >> 1;
     float* cs = sm;                         // [half]
     float* sn = cs + half;                  // [half]
@@ -66,24 +67,21 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a) {
     const int qw = a.dn + a.rd;
     if (a.q_full) {                          // whole heads for a kernel that scores expanded keys: [unrotated | rotated]
         T* qf = (T*)a.q_full + (size_t)t * a.qf_stride;
-        for (int i = threadIdx.x; i < a.H * qw; i += blockDim.x) {
-            const int h = i / qw, d = i % qw;
-            stf(qf + i, d < a.dn ? row[i] : rotated(row + h * qw + a.dn, d - a.dn, a.rope, cs, sn));
-        }
+        for (int h = h0; h < a.H; h += h_step)
+            for (int d = threadIdx.x; d < qw; d += blockDim.x)
+                stf(qf + h * qw + d, d < a.dn ? row[h * qw + d] : rotated(row + h * qw + a.dn, d - a.dn, a.rope, cs, sn));
     } else {
         T* qn = (T*)a.q_nope + (size_t)t * a.qn_stride;
         T* qa = (T*)a.q_abs + (size_t)t * a.qa_stride;
-        for (int i = threadIdx.x; i < a.H * a.dn; i += blockDim.x) {
-            const int h = i / a.dn, d = i % a.dn;
-            stf(qn + i, row[h * qw + d]);
-        }
         const int tail = a.dk - a.r;        // rotated part and padding
-        for (int i = threadIdx.x; i < a.H * tail; i += blockDim.x) {
-            const int h = i / tail, e = i % tail;
-            stf(qa + (size_t)h * a.dk + a.r + e, e < a.rd ? rotated(row + h * qw + a.dn, e, a.rope, cs, sn) : 0.f);
-        }
+        for (int h = h0; h < a.H; h += h_step)
+            for (int d = threadIdx.x; d < a.dn + tail; d += blockDim.x) {
+                const int e = d - a.dn;
+                if (e < 0) stf(qn + h * a.dn + d, row[h * qw + d]);
+                else stf(qa + (size_t)h * a.dk + a.r + e, e < a.rd ? rotated(row + h * qw + a.dn, e, a.rope, cs, sn) : 0.f);
+            }
     }
-    if (!a.owner) return;
+    if (!a.owner || h0 != 0) return;
     const float* lat = a.kv_in ? a.kv_in + (size_t)t * a.in_stride : row + a.H * qw;
     float ss = 0.f;
     for (int i = threadIdx.x; i < a.r; i += blockDim.x) ss += lat[i] * lat[i];
@@ -129,8 +127,10 @@ extern "C" int tb_latent_prep(const LatentArgs* args, int out_dtype, cudaStream_
     TB_REQUIRE(!a.owner || a.latent_w, "latent_prep: the latent's norm weight is missing");
     TB_REQUIRE(!a.append || (a.owner && a.cache.storage && a.cache.head_dim == a.dk && a.cache.kv_heads == 1), "latent_prep: the cache view does not match the rows");
     const size_t smem = (size_t)(a.rope.rot + 2) * sizeof(float);
-    if (out_dtype == TB_F32) tb_launch(latent_prep_kernel<float>, a.T, 128, smem, stream, a);
-    else if (out_dtype == TB_BF16) tb_launch(latent_prep_kernel<__nv_bfloat16>, a.T, 128, smem, stream, a);
+    const int parts = a.T >= 592 ? 1 : (a.T >= 148 ? (a.H < 4 ? a.H : 4) : (a.H < 32 ? a.H : 32));      // a block a head while tokens are few
+    const dim3 grid(a.T, parts);
+    if (out_dtype == TB_F32) tb_launch(latent_prep_kernel<float>, grid, 128, smem, stream, a);
+    else if (out_dtype == TB_BF16) tb_launch(latent_prep_kernel<__nv_bfloat16>, grid, 128, smem, stream, a);
     else TB_REQUIRE(false, "latent_prep: unknown dtype %d", out_dtype);
     TB_CHECK_LAUNCH("latent_prep");
     return 0;

@@ -40,14 +40,27 @@ __global__ void __launch_bounds__(256) polynorm_kernel(const T* z, int ldz, cons
     }
 }
 
-template <typename T, typename G>
+// V neighbouring elements a thread (4 where rows, strides and width allow accesses of four elements).
+template <typename T, typename G, int V>
 __global__ void __launch_bounds__(256) gate_rows_kernel(const T* x, int ldx, const G* __restrict__ g, int ldg,
                                                         T* y, int ldy, int n, int act, float scale) {
     pdl_launch_dependents();
     pdl_wait();
     const size_t t = blockIdx.y;
-    const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < n) stf(y + t * ldy + i, ldf(x + t * ldx + i) * act_gate(ldf(g + t * ldg + i), act) * scale);
+    if (V == 1) {
+        const int i = blockIdx.x * blockDim.x + threadIdx.x;
+        if (i < n) stf(y + t * ldy + i, ldf(x + t * ldx + i) * act_gate(ldf(g + t * ldg + i), act) * scale);
+        return;
+    }
+    struct alignas(sizeof(T) * V) VT { T v[V]; };
+    struct alignas(sizeof(G) * V) VG { G v[V]; };
+    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+    if (i >= n) return;
+    VT o = *reinterpret_cast<const VT*>(x + t * ldx + i);
+    const VG gate = *reinterpret_cast<const VG*>(g + t * ldg + i);
+#pragma unroll
+    for (int e = 0; e < V; ++e) stf(o.v + e, ldf(o.v + e) * act_gate(ldf(gate.v + e), act) * scale);
+    *reinterpret_cast<VT*>(y + t * ldy + i) = o;
 }
 
 template <typename T, typename G>
@@ -81,10 +94,14 @@ extern "C" int tb_polynorm(const void* z, int ldz, const float* coef, float eps,
 
 template <typename T, typename G>
 static void launch_gate_rows(const void* x, int ldx, const void* g, int ldg, void* y, int ldy, int rows, int n, int act, float scale, cudaStream_t stream) {
+    const bool four = n % 4 == 0 && ldx % 4 == 0 && ldg % 4 == 0 && ldy % 4 == 0 && (((uintptr_t)x | (uintptr_t)g | (uintptr_t)y) & 15) == 0;
     for (int r0 = 0; r0 < rows; r0 += 65535) {
         const int nr = rows - r0 < 65535 ? rows - r0 : 65535;
-        tb_launch(gate_rows_kernel<T, G>, dim3((n + 255) / 256, nr), dim3(256), 0, stream, (const T*)x + (size_t)r0 * ldx, ldx, (const G*)g + (size_t)r0 * ldg, ldg,
-                  (T*)y + (size_t)r0 * ldy, ldy, n, act, scale);
+        const T* xr = (const T*)x + (size_t)r0 * ldx;
+        const G* gr = (const G*)g + (size_t)r0 * ldg;
+        T* yr = (T*)y + (size_t)r0 * ldy;
+        if (four) tb_launch(gate_rows_kernel<T, G, 4>, dim3((n / 4 + 255) / 256, nr), dim3(256), 0, stream, xr, ldx, gr, ldg, yr, ldy, n, act, scale);
+        else tb_launch(gate_rows_kernel<T, G, 1>, dim3((n + 255) / 256, nr), dim3(256), 0, stream, xr, ldx, gr, ldg, yr, ldy, n, act, scale);
     }
 }
 

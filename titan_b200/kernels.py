@@ -309,6 +309,8 @@ def alib():
         l = _build.load("attention")
         l.tb_attn_decode_mma.argtypes = [POINTER(AttnArgs), c_void_p]
         l.tb_attn_decode_mma_check.argtypes = [POINTER(AttnArgs), c_int]
+        l.tb_attn_decode_latent.argtypes = [POINTER(AttnArgs), c_void_p]
+        l.tb_attn_decode_latent_check.argtypes = [POINTER(AttnArgs), c_int]
         l.tb_attn_prefill_mma.argtypes = [POINTER(AttnArgs), c_int, c_void_p]
         l.tb_attn_prefill_mma_check.argtypes = [POINTER(AttnArgs), c_int, c_int]
         l.tb_attn_prefill_split.argtypes = [POINTER(SplitAttnArgs), c_void_p]
@@ -890,6 +892,15 @@ def attn_decode_mma(args: AttnArgs, stream: int) -> None:
     _check(alib().tb_attn_decode_mma(byref(args), stream))
 
 
+def attn_decode_latent_accepts(args: AttnArgs, dtype: torch.dtype) -> bool:
+    return dtype == torch.bfloat16 and alib().tb_attn_decode_latent_check(byref(args), BF16) == 0
+
+
+def attn_decode_latent(args: AttnArgs, stream: int) -> None:
+    """Decode attention over a shared latent on tensor cores (bfloat16, one row a token as key and value), then the merge of the splits."""
+    _check(alib().tb_attn_decode_latent(byref(args), stream))
+
+
 def set_attn_decode_cluster(on: bool) -> None:
     """Decode attention with up to 16 splits: merge them inside a thread-block cluster (on by default) or through
     scratch memory and the merge kernel."""
@@ -976,7 +987,7 @@ def wait_errors() -> dict:
         return {}
     found = {"gemm_tc": gemm_tc_error()}
     if _alib is not None:
-        found.update({"attn_prefill_tc": attn_tc_error(), "attn_mma": attn_mma_error()})
+        found.update({"attn_prefill_tc": attn_tc_error(), "attn_mma": attn_mma_error(), "attn_decode_latent": int(alib().tb_attn_latent_error())})
     return {k: v for k, v in found.items() if v}
 
 

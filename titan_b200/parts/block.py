@@ -394,7 +394,7 @@ class SandwichBlock(Part):
     in a step of single tokens that is the sequence's state, so the same kernel shifts too; in a step of longer runs the next
     block's own kernel norms and shifts (the row before is a neighbour's).  The previous token's normed row, before its own
     shift, is the block's state: float32, one row a sequence and run, in a ``state`` cache group (zero at a sequence's start).
-    The rows X_j live in a buffer of the step ([runs, T, W] float32): nothing of them outlasts it."""
+    The rows X_j live in one scratch buffer ([runs, T, W] float32); none of them outlasts its step."""
 
     def __init__(self, spec):
         if spec.mixer_norm is None or (spec.feed_forward is None) != (spec.feed_forward_norm is None) or len(spec.norms) != (1 if spec.feed_forward is None else 2):
@@ -476,7 +476,10 @@ class SandwichBlock(Part):
                 raise RuntimeError(f"a block with {self.place + 2} depth weights runs as number {ctx.run}")
             history = ctx.carried.get("depth_rows")
             if ctx.run == 0:                                              # the rows that enter the first block are depth 0: its first join keeps them
-                history = ctx.carried["depth_rows"] = ctx.empty((ctx.runs,) + tuple(x.shape), torch.float32)
+                held, n = ctx.scratch.get("depth_rows"), ctx.runs * x.numel()
+                if held is None or held.numel() < n:                      # kept from step to step: as large as the longest one so far
+                    held = ctx.scratch["depth_rows"] = ctx.empty((n,), torch.float32)
+                history = ctx.carried["depth_rows"] = held[:n].view((ctx.runs,) + tuple(x.shape))
                 keep = history[0]
             elif history is None:
                 raise RuntimeError("an average over depth needs every block from the first on to keep its rows")

@@ -250,21 +250,30 @@ class LatentAttentionMixer(Mixer):
         aa.window, aa.scale = s.window or 0, self.scale
         aa.sink = None if self.sink is None else self.sink.data_ptr()
         if decode:
-            # all heads read one row per key: a block for every few heads (not one for the single "kv head"), and splits
-            # of one page, or of half a page while that still leaves SMs without a block (a step of one or two sequences:
-            # measured at 16 heads and a window of 1,024, 0.61 -> 0.56 ms a step at batch 1, 0.87 -> 0.88 at batch 8)
-            aa.head_blocks = H // 4 if H % 4 == 0 else (H // 2 if H % 2 == 0 else H)          # four heads (a warp each), two, or one a block
-            span = min(s.window or lay.max_kv_len, lay.max_kv_len)
-            few = lay.B * aa.head_blocks * -(-span // 64) < int(ctx.options.get("sm_count", 148))
-            chunk = int(ctx.options.get("latent_chunk", 32 if few else 64))
-            chunk, splits = decode_split(lay, 1, dict(ctx.options, attn_chunk=chunk), False)
-            need = lay.B * H * splits * (r + 2)
-            scratch = ctx.scratch.get("attn_partials")
-            if scratch is None or scratch.numel() < need:
-                scratch = ctx.scratch["attn_partials"] = torch.empty(need, dtype=torch.float32, device=ctx.device)
             aa.kv_new, aa.kv_stride = None, 0
-            aa.chunk, aa.n_splits, aa.scratch = chunk, splits, scratch.data_ptr()
-            K.attn_decode(aa, q_abs.dtype, ctx.stream)
+            fast = ctx.dtype == torch.bfloat16 and ctx.options.get("attention", "fast") != "plain"
+            if fast:
+                # tensor cores: sixteen heads a block, splits of one page while they do not fill the machine (a block an SM), at most 64
+                sms = int(ctx.options.get("sm_count", 148))
+                chunk, splits = 64, max(1, min(64, sms // (lay.B * -(-H // 16))))
+                self._decode_scratch(aa, ctx, chunk, splits)
+                if ctx.options.get("early_pages", True):       # lengths the kernel may read before its predecessors end
+                    if lay.lengths_by_copy:
+                        aa.early_len, aa.early_mode = lay.kv_len.data_ptr(), 1
+                    elif lay.committed_len is not None:
+                        aa.early_len, aa.early_mode = lay.committed_len.data_ptr(), 2
+            if fast and K.attn_decode_latent_accepts(aa, ctx.dtype):
+                K.attn_decode_latent(aa, ctx.stream)
+            else:
+                # all heads read one row per key: a block for every few heads (not one for the single "kv head"), and splits
+                # of one page, or of half a page while that still leaves SMs without a block (a step of one or two sequences:
+                # measured at 16 heads and a window of 1,024, 0.61 -> 0.56 ms a step at batch 1, 0.87 -> 0.88 at batch 8)
+                aa.head_blocks = H // 4 if H % 4 == 0 else (H // 2 if H % 2 == 0 else H)          # four heads (a warp each), two, or one a block
+                span = min(s.window or lay.max_kv_len, lay.max_kv_len)
+                few = lay.B * aa.head_blocks * -(-span // 64) < int(ctx.options.get("sm_count", 148))
+                chunk = int(ctx.options.get("latent_chunk", 32 if few else 64))
+                self._decode_scratch(aa, ctx, *decode_split(lay, 1, dict(ctx.options, attn_chunk=chunk), False))
+                K.attn_decode(aa, q_abs.dtype, ctx.stream)
         else:
             aa.kv_new, aa.kv_stride = rows.data_ptr(), rows.stride(0)
             K.attn_prefill(aa, q_abs.dtype, ctx.stream)
@@ -273,6 +282,13 @@ class LatentAttentionMixer(Mixer):
         linear.matmul_heads(lat, self.w_uv, o, H, r, dv, ctx)
         self._gate(o, h, proj, ctx)
         linear.matmul(o, self.w_o, out, linear.EPI_ADD, ctx)
+
+    def _decode_scratch(self, aa: K.AttnArgs, ctx, chunk: int, splits: int) -> None:
+        need = ctx.layout.B * self.H * splits * (self.r + 2)
+        scratch = ctx.scratch.get("attn_partials")
+        if scratch is None or scratch.numel() < need:
+            scratch = ctx.scratch["attn_partials"] = torch.empty(need, dtype=torch.float32, device=ctx.device)
+        aa.chunk, aa.n_splits, aa.scratch = chunk, splits, scratch.data_ptr()
 
     def _gate(self, o: torch.Tensor, h, proj: torch.Tensor, ctx) -> None:
         """The concatenated heads times sigmoid(W_g h), in place, where the layer has such a gate."""
