@@ -27,8 +27,15 @@ struct PairPrepArgs {
 
 namespace {
 
+__device__ __forceinline__ void store_four(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store_four(__nv_bfloat16* p, const float4& v) {
+    alignas(8) __nv_bfloat16 t[4];
+    stf(t, v.x); stf(t + 1, v.y); stf(t + 2, v.z); stf(t + 3, v.w);
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(t);
+}
+
 // A warp takes one piece of a token: a map of a query head, a map of a key head, or a value head.
-template <typename T>
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256) pair_prep_kernel(PairPrepArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -45,9 +52,17 @@ __global__ void __launch_bounds__(256) pair_prep_kernel(PairPrepArgs a) {
     float scale = 1.f;
     if (w) {
         float ss = 0.f;
-        for (int e = lane; e < n; e += 32) {
-            const float v = src[e] + (bias ? bias[e] : 0.f);
-            ss = fmaf(v, v, ss);
+        if (VEC) {
+            for (int e = lane * 4; e < n; e += 128) {
+                float4 v = *reinterpret_cast<const float4*>(src + e);
+                if (bias) { const float4 c = *reinterpret_cast<const float4*>(bias + e); v.x += c.x; v.y += c.y; v.z += c.z; v.w += c.w; }
+                ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            }
+        } else {
+            for (int e = lane; e < n; e += 32) {
+                const float v = src[e] + (bias ? bias[e] : 0.f);
+                ss = fmaf(v, v, ss);
+            }
         }
         scale = 1.0f / sqrtf(warp_sum(ss) / (float)n + a.eps);
     }
@@ -62,6 +77,24 @@ __global__ void __launch_bounds__(256) pair_prep_kernel(PairPrepArgs a) {
         const int head = is_v ? piece - nq - nk : (piece - nq) >> 1;
         if (a.kv_out) own = (T*)a.kv_out + (size_t)t * a.kv_stride + (size_t)(is_v ? a.G + head : head) * a.hd;
         if (a.append) page = (T*)a.cache.storage + (is_v ? kv_half_elems(a.cache) : 0) + kv_row_offset(a.cache, a.slot_of_seq[a.seq_of[t]], a.pos_of[t], head);
+    }
+    if (VEC) {
+        // four neighbouring elements a lane
+        for (int i = lo + lane * 4; i < hi; i += 128) {
+            const int e = i - at;
+            float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (e >= 0 && e < n) {
+                v = *reinterpret_cast<const float4*>(src + e);
+                if (bias) { const float4 c = *reinterpret_cast<const float4*>(bias + e); v.x += c.x; v.y += c.y; v.z += c.z; v.w += c.w; }
+                if (w) {
+                    const float4 c = *reinterpret_cast<const float4*>(w + e);
+                    v.x = v.x * scale * c.x; v.y = v.y * scale * c.y; v.z = v.z * scale * c.z; v.w = v.w * scale * c.w;
+                }
+            }
+            if (own) store_four(own + i, v);
+            if (page) store_four(page + i, v);
+        }
+        return;
     }
     for (int i = lo + lane; i < hi; i += 32) {
         const int e = i - at;
@@ -126,8 +159,15 @@ extern "C" int tb_pair_prep(const PairPrepArgs* args, int dtype, cudaStream_t st
     const int pieces = 2 * a.H + 3 * a.G, warps = 8;
     TB_REQUIRE((pieces + warps - 1) / warps <= 65535, "pair_prep: too many heads");
     const dim3 grid(a.T, (pieces + warps - 1) / warps);
-    if (dtype == TB_F32) tb_launch(pair_prep_kernel<float>, grid, warps * 32, 0, stream, a);
-    else if (dtype == TB_BF16) tb_launch(pair_prep_kernel<__nv_bfloat16>, grid, warps * 32, 0, stream, a);
+    const bool vec = a.dim % 4 == 0 && a.vdim % 4 == 0 && a.hd % 4 == 0 && a.in_stride % 4 == 0 && a.q_stride % 4 == 0 && a.kv_stride % 4 == 0 &&
+                     (((uintptr_t)a.in | (uintptr_t)a.bias | (uintptr_t)a.q_w | (uintptr_t)a.k_w | (uintptr_t)a.q_out | (uintptr_t)a.kv_out | (uintptr_t)a.cache.storage) & 15) == 0;
+    if (dtype == TB_F32) {
+        if (vec) tb_launch(pair_prep_kernel<float, true>, grid, warps * 32, 0, stream, a);
+        else tb_launch(pair_prep_kernel<float, false>, grid, warps * 32, 0, stream, a);
+    } else if (dtype == TB_BF16) {
+        if (vec) tb_launch(pair_prep_kernel<__nv_bfloat16, true>, grid, warps * 32, 0, stream, a);
+        else tb_launch(pair_prep_kernel<__nv_bfloat16, false>, grid, warps * 32, 0, stream, a);
+    }
     else TB_REQUIRE(false, "pair_prep: unknown dtype %d", dtype);
     TB_CHECK_LAUNCH("pair_prep");
     return 0;

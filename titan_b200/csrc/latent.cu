@@ -42,7 +42,16 @@ __device__ __forceinline__ float rotated(const float* x, int e, const TbRotary& 
     return x[e] * cs[k] + sign * x[partner] * sn[k];
 }
 
-template <typename T>
+__device__ __forceinline__ void put4(float* p, const float* v) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void put4(__nv_bfloat16* p, const float* v) {
+    alignas(8) __nv_bfloat16 t[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) stf(t + i, v[i]);
+    *reinterpret_cast<uint2*>(p) = *reinterpret_cast<const uint2*>(t);
+}
+
+// V: neighbouring elements a thread takes at a time (4 where every width, stride and address allows it).
+template <typename T, int V>
 __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a) {
     pdl_launch_dependents();
     pdl_wait();
@@ -67,14 +76,45 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(LatentArgs a) {
     const int qw = a.dn + a.rd;
     if (a.q_full) {                          // whole heads for a kernel that scores expanded keys: [unrotated | rotated]
         T* qf = (T*)a.q_full + (size_t)t * a.qf_stride;
-        for (int h = h0; h < a.H; h += h_step)
+        if (V == 4) {
+            const int per = qw / 4, n = ((a.H - h0 + h_step - 1) / h_step) * per;
+            for (int i = threadIdx.x; i < n; i += blockDim.x) {
+                const int h = h0 + (i / per) * h_step, d = (i % per) * 4;
+                const float* src = row + h * qw;
+                float v[4];
+                if (d < a.dn) {
+                    const float4 f = *reinterpret_cast<const float4*>(src + d);
+                    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v[e] = rotated(src + a.dn, d - a.dn + e, a.rope, cs, sn);
+                }
+                put4(qf + h * qw + d, v);
+            }
+        } else for (int h = h0; h < a.H; h += h_step)
             for (int d = threadIdx.x; d < qw; d += blockDim.x)
                 stf(qf + h * qw + d, d < a.dn ? row[h * qw + d] : rotated(row + h * qw + a.dn, d - a.dn, a.rope, cs, sn));
     } else {
         T* qn = (T*)a.q_nope + (size_t)t * a.qn_stride;
         T* qa = (T*)a.q_abs + (size_t)t * a.qa_stride;
         const int tail = a.dk - a.r;        // rotated part and padding
-        for (int h = h0; h < a.H; h += h_step)
+        if (V == 4) {
+            const int per = (a.dn + tail) / 4, n = ((a.H - h0 + h_step - 1) / h_step) * per;
+            for (int i = threadIdx.x; i < n; i += blockDim.x) {
+                const int h = h0 + (i / per) * h_step, d = (i % per) * 4, e0 = d - a.dn;
+                const float* src = row + h * qw;
+                float v[4];
+                if (e0 < 0) {
+                    const float4 f = *reinterpret_cast<const float4*>(src + d);
+                    v[0] = f.x; v[1] = f.y; v[2] = f.z; v[3] = f.w;
+                    put4(qn + h * a.dn + d, v);
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) v[e] = e0 + e < a.rd ? rotated(src + a.dn, e0 + e, a.rope, cs, sn) : 0.f;
+                    put4(qa + (size_t)h * a.dk + a.r + e0, v);
+                }
+            }
+        } else for (int h = h0; h < a.H; h += h_step)
             for (int d = threadIdx.x; d < a.dn + tail; d += blockDim.x) {
                 const int e = d - a.dn;
                 if (e < 0) stf(qn + h * a.dn + d, row[h * qw + d]);
@@ -129,8 +169,15 @@ extern "C" int tb_latent_prep(const LatentArgs* args, int out_dtype, cudaStream_
     const size_t smem = (size_t)(a.rope.rot + 2) * sizeof(float);
     const int parts = a.T >= 592 ? 1 : (a.T >= 148 ? (a.H < 4 ? a.H : 4) : (a.H < 32 ? a.H : 32));      // a block a head while tokens are few
     const dim3 grid(a.T, parts);
-    if (out_dtype == TB_F32) tb_launch(latent_prep_kernel<float>, grid, 128, smem, stream, a);
-    else if (out_dtype == TB_BF16) tb_launch(latent_prep_kernel<__nv_bfloat16>, grid, 128, smem, stream, a);
+    const bool four = a.dn % 4 == 0 && a.rd % 4 == 0 && a.r % 4 == 0 && a.in_stride % 4 == 0 && a.qn_stride % 4 == 0 && a.qa_stride % 4 == 0 && a.qf_stride % 4 == 0 &&
+                      (((uintptr_t)a.in | (uintptr_t)a.q_nope | (uintptr_t)a.q_abs | (uintptr_t)a.q_full) & 15) == 0;
+    if (out_dtype == TB_F32) {
+        if (four) tb_launch(latent_prep_kernel<float, 4>, grid, 128, smem, stream, a);
+        else tb_launch(latent_prep_kernel<float, 1>, grid, 128, smem, stream, a);
+    } else if (out_dtype == TB_BF16) {
+        if (four) tb_launch(latent_prep_kernel<__nv_bfloat16, 4>, grid, 128, smem, stream, a);
+        else tb_launch(latent_prep_kernel<__nv_bfloat16, 1>, grid, 128, smem, stream, a);
+    }
     else TB_REQUIRE(false, "latent_prep: unknown dtype %d", out_dtype);
     TB_CHECK_LAUNCH("latent_prep");
     return 0;
