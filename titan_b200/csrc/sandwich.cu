@@ -263,7 +263,8 @@ int launch_join(const SandwichArgs& a, cudaStream_t stream) {
         return 0;
     }
     // a few rows: many threads a row, one vector each; many rows: two or four vectors a thread, so that more rows are in flight
-    const int n4 = a.W / 4, per = a.rows <= 296 ? 1 : (n4 >= 512 ? 4 : 2);
+    // (two where the history is read as well: its sums take registers)
+    const int n4 = a.W / 4, per = a.rows <= 296 ? 1 : (n4 >= 512 && a.n_hist == 0 ? 4 : 2);
     int threads = threads_for((n4 + per - 1) / per);
     const int held = (n4 + threads - 1) / threads;
     if (held <= 1) tb_launch(sandwich_join_kernel<T, 4, 1>, a.rows, threads, 0, stream, a);
@@ -304,7 +305,7 @@ extern "C" int tb_shift_norm(const ShiftNormArgs* args, int h_dtype, cudaStream_
     ShiftNormArgs a = *args;
     TB_REQUIRE(a.rows > 0 && a.W > 0 && a.x && a.w && a.mu && a.h, "shift_norm: rows, the norm's weight and the shift's factors are wanted");
     TB_REQUIRE(a.state && a.state_stride >= a.W && a.seq_of && a.q_start && a.slot_of_seq, "shift_norm: the sequences' states are wanted");
-    if (a.rows_per_block <= 0) a.rows_per_block = a.rows >= 1184 ? 4 : 1;
+    if (a.rows_per_block <= 0) a.rows_per_block = a.rows >= 592 ? 2 : 1;
     if (h_dtype == TB_F32) launch_shift<float>(a, stream);
     else if (h_dtype == TB_BF16) launch_shift<__nv_bfloat16>(a, stream);
     else TB_REQUIRE(false, "shift_norm: unknown dtype %d", h_dtype);
