@@ -749,3 +749,28 @@ def test_configurations_drawn_at_random(seed, dtype):
             continue
         rows = (got.double() - want.double()).norm(dim=1) / want.double().norm(dim=1)
         assert float(rows.median()) < 3 * TOL[dtype] and float((rows > 12 * TOL[dtype]).double().mean()) <= 0.1, f"seed {seed}: {what}: {float(rows.median()):.3f} {float(rows.max()):.3f}"
+
+
+def test_a_steps_context_is_freed_with_its_last_reference():
+    """Nothing of a step refers back to its context: the step's buffers go back to the allocator when the step returns, not when
+    Python's cycle collector next runs (prompts would otherwise take new device memory step after step)."""
+    import gc
+    import weakref
+    from titan_b200 import StepEntry
+    wd = world("mix")
+    e = wd.engine("bfloat16")
+    made = []
+    real = e._context
+    e._context = lambda layout: (lambda ctx: (made.append(weakref.ref(ctx)), ctx)[1])(real(layout))
+    was = gc.isenabled()
+    gc.disable()
+    try:
+        s = e.alloc_slot()
+        e.step([StepEntry(s, wd.requests[0], [0])])
+        e.step([StepEntry(s, [1], [0])])
+        e.free_slot(s)
+        assert len(made) == 2 and all(r() is None for r in made), "a step's context outlives the step"
+    finally:
+        del e._context
+        if was:
+            gc.enable()

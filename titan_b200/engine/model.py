@@ -92,8 +92,8 @@ class DecoderModel:
             x = x.repeat(1, streams)
         if "row_sums" not in ctx.scratch:      # places where folded norms leave sums of squares: one per run of a layer
             ctx.scratch["row_sums"] = torch.zeros((len(self.spec.order), 16, 32), dtype=torch.float32, device=ctx.device)
-        ctx.runs = len(self.spec.order)
-        ctx.block_state = lambda run: cache.view_for_layer(ctx.runs + run)
+        ctx.runs = runs = len(self.spec.order)
+        ctx.block_state = lambda run: cache.view_for_layer(runs + run)      # (holds no reference to ctx: a cycle would keep the step's tensors until the collector runs)
         for run, i in enumerate(self.spec.order):
             ctx.run = run
             ctx.next_block = self.blocks[self.spec.order[run + 1]] if run + 1 < len(self.spec.order) else None
