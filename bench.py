@@ -670,7 +670,7 @@ def launcher_times(engine, torch, K, entries):
                          "attn_prefill_mma", "attn_prefill_tc", "attn_prefill_split", "moe_gather", "latent_prep", "latent_append", "lightning_scan", "lightning_chunks",
                          "gated_rmsnorm", "moe_route", "token_gate_rows", "moe_plan", "moe_grouped", "moe_rows", "moe_combine", "moe_experts_tc",
                          "dyt", "scale_add", "wkv", "moe_route_all", "hyper", "polynorm", "gate_rows", "head_norm_gate", "delta_prep",
-                         "recurrent_scan", "group_rmsnorm", "residual_group_norm", "qkv_whole_norm", "attn_mixed_prefill", "attn_mixed_decode",
+                         "recurrent_scan", "group_rmsnorm", "residual_group_norm", "qkv_whole_norm", "attn_mixed_prefill", "attn_mixed_decode", "attn_decode_latent",
                          "rotary_rows", "moe_route_scored", "pair_prep", "pair_combine", "sandwich_join", "shift_norm") if hasattr(K, n)]
     events, originals = [], {n: getattr(K, n) for n in names}
 
