@@ -37,6 +37,9 @@ class PositionSpec:
     rotary_dim: int = 0       # leading dims of a head that are rotated
     theta: float = 10000.0
     pairing: str = "half"     # "half": (k, k + rotary_dim/2) turn together; "adjacent": (2k, 2k + 1)
+    # Frequencies scaled by wavelength (the rule of Llama 3.1): (factor, low, high, original).  Waves shorter than original / high stay,
+    # waves longer than original / low turn factor times slower, and between the two the frequency is a blend.  None: as they are.
+    scaling: Optional[Tuple[float, float, float, float]] = None
 
 
 def _lookup(pairs, key, default):
@@ -112,6 +115,27 @@ class LayerSpec:
 
 
 @dataclass(frozen=True)
+class LoopSpec:
+    """A stretch of layers, start .. stop - 1, that runs ``times`` times in a row with the same weights; every pass has caches of
+    its own.  Before the first layer of pass t (the first pass too): x <- W [x ; x0], x0 the rows that entered the first layer
+    (``mix``: name of W [H, 2 H], x first; None: x stays), then x <- x + S[t] (``step``: name of S [times, H]; None: nothing)."""
+    start: int
+    stop: int
+    times: int
+    mix: Optional[str] = None
+    step: Optional[str] = None
+
+    def order(self, layers: int) -> Tuple[int, ...]:
+        """The running order of a model of ``layers`` layers."""
+        return tuple(range(self.start)) + tuple(range(self.start, self.stop)) * self.times + tuple(range(self.stop, layers))
+
+    def pass_at(self, run: int) -> Optional[int]:
+        """The number of the pass that begins right before run ``run`` of the order; None if none does."""
+        t, inside = divmod(run - self.start, self.stop - self.start)
+        return t if inside == 0 and 0 <= t < self.times else None
+
+
+@dataclass(frozen=True)
 class ModelSpec:
     architecture: str
     hidden_size: int
@@ -133,6 +157,7 @@ class ModelSpec:
     # Tensors that a file of this model may hold although the model, as described, uses none of them (the factor of a
     # mechanism that a layer's description switches off): present or absent, they are not an error and are not loaded.
     ignorable_tensors: Tuple[str, ...] = ()
+    loop: Optional[LoopSpec] = None       # what stands before the passes of a repeated stretch of layers; ``order`` is then loop.order(len(layers))
 
     def validate(self) -> None:
         if not self.layers:
@@ -140,6 +165,14 @@ class ModelSpec:
         for i in self.order:
             if not 0 <= i < len(self.layers):
                 raise ConfigError(f"layer order names layer {i}, but there are {len(self.layers)} layers")
+        if self.loop is not None:
+            p = self.loop
+            if not 0 <= p.start < p.stop <= len(self.layers) or p.times < 1:
+                raise ConfigError(f"a loop over layers {p.start} .. {p.stop - 1}, {p.times} times, in a model of {len(self.layers)} layers")
+            if self.order != p.order(len(self.layers)):
+                raise ConfigError("the running order is not that of the loop")
+            if self.streams > 1:
+                raise ConfigError("a loop's entry works on one residual stream")
         if self.streams < 1 or (self.streams > 1 and any(l.arrangement != "hyper" for l in self.layers)):
             raise ConfigError(f"{self.streams} residual streams need every block to be of the 'hyper' arrangement")
         for layer in self.layers:

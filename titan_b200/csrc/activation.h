@@ -12,8 +12,18 @@
 #define TB_ACT_GELU_TANH 1
 #define TB_ACT_SWISH_CLAMPED 2
 #define TB_ACT_KINDS 3
+// Activations of one sum (a feed-forward without a gate), for the STORE epilogue; they travel in the same ``act``:
+//
+//   TB_UNARY_NONE         z                       TB_UNARY_RELU2   max(z, 0)^2
+#define TB_UNARY_NONE 0
+#define TB_UNARY_RELU2 1
+#define TB_UNARY_KINDS 2
 
 #ifdef __CUDACC__
+__device__ __forceinline__ float tb_unary(int act, float z) {
+    const float r = fmaxf(z, 0.f);
+    return act == TB_UNARY_RELU2 ? r * r : z;
+}
 __device__ __forceinline__ float tb_gated(int act, float limit, float g, float u) {
     if (act == TB_ACT_GELU_TANH) {
         const float inner = 0.7978845608028654f * (g + 0.044715f * g * g * g);

@@ -7,7 +7,7 @@
 // fuse the residual into the epilogue (:3489-3493) and SwiGLU into gate/up (:2589).
 //
 // Epilogues:
-//   TB_EPI_STORE   out[m][n] = acc                      (compute dtype)
+//   TB_EPI_STORE   out[m][n] = acc                      (compute dtype), or an activation of it (activation.h)
 //   TB_EPI_F32     out[m][n] = acc                      (float32: logits)
 //   TB_EPI_ADD     out[m][n] += acc                     (float32 residual stream, in place)
 //   TB_EPI_SWIGLU  out[m][j] = gate(acc[2j], acc[2j+1]) (rows of W interleaved gate, up; N even); the gate is
@@ -84,7 +84,7 @@ gemm_simt_kernel(const T* __restrict__ X, const T* __restrict__ W, void* __restr
             for (int j = 0; j < TN; ++j) {
                 const int n = n0 + tx * TN + j;
                 if (n >= N) continue;
-                if (EPI == TB_EPI_STORE) stf((T*)out + (size_t)m * ldo + n, acc[i][j]);
+                if (EPI == TB_EPI_STORE) stf((T*)out + (size_t)m * ldo + n, tb_unary(act, acc[i][j]));
                 if (EPI == TB_EPI_F32) ((float*)out)[(size_t)m * ldo + n] = acc[i][j];
                 if (EPI == TB_EPI_ADD) ((float*)out)[(size_t)m * ldo + n] += acc[i][j];
             }
@@ -113,7 +113,7 @@ int launch(const void* X, const void* W, void* out, int M, int N, int K, int ldx
 template <typename T, int EPI>
 __global__ void __launch_bounds__(256)
 gemm_rows_kernel(const T* __restrict__ X, const T* __restrict__ W, void* __restrict__ out_, int M, int N, int K, int ldx, int ldo,
-                 long long sx, long long sw, long long so) {
+                 long long sx, long long sw, long long so, int act) {
     pdl_launch_dependents();
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -144,20 +144,20 @@ gemm_rows_kernel(const T* __restrict__ X, const T* __restrict__ W, void* __restr
     acc = warp_sum(acc);
     if (lane != 0) return;
     const size_t at = (size_t)z * so + (size_t)m * ldo + n;
-    if (EPI == TB_EPI_STORE) stf((T*)out_ + at, acc);
+    if (EPI == TB_EPI_STORE) stf((T*)out_ + at, tb_unary(act, acc));
     if (EPI == TB_EPI_F32) ((float*)out_)[at] = acc;
     if (EPI == TB_EPI_ADD) ((float*)out_)[at] += acc;
 }
 
 template <typename T>
 static int launch_rows(const void* X, const void* W, void* out, int M, int N, int K, int ldx, int ldo, int epi, int batch,
-                       long long sx, long long sw, long long so, cudaStream_t stream) {
+                       long long sx, long long sw, long long so, int act, cudaStream_t stream) {
     dim3 grid((N + 7) / 8, M, batch);
     const T* x = (const T*)X;
     const T* w = (const T*)W;
-    if (epi == TB_EPI_STORE) tb_launch(gemm_rows_kernel<T, TB_EPI_STORE>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so);
-    else if (epi == TB_EPI_F32) tb_launch(gemm_rows_kernel<T, TB_EPI_F32>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so);
-    else if (epi == TB_EPI_ADD) tb_launch(gemm_rows_kernel<T, TB_EPI_ADD>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so);
+    if (epi == TB_EPI_STORE) tb_launch(gemm_rows_kernel<T, TB_EPI_STORE>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so, act);
+    else if (epi == TB_EPI_F32) tb_launch(gemm_rows_kernel<T, TB_EPI_F32>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so, act);
+    else if (epi == TB_EPI_ADD) tb_launch(gemm_rows_kernel<T, TB_EPI_ADD>, grid, 256, 0, stream, x, w, out, M, N, K, ldx, ldo, sx, sw, so, act);
     else { tb_set_error("gemm_rows: epilogue %d is not one of store, float32, add", epi); return 1; }
     return 0;
 }
@@ -166,11 +166,11 @@ static int launch_rows(const void* X, const void* W, void* out, int M, int N, in
 
 // ldx: row stride of X in elements; ldo: row stride of out in elements.  ``batch`` products of the same shape in one
 // launch: product z reads X + z * sx and W + z * sw and writes out + z * so (offsets in elements).
-// act, limit: the gate of the SWIGLU epilogue (activation.h).
+// act, limit: the gate of the SWIGLU epilogue, or the activation of the STORE epilogue (activation.h).
 extern "C" int tb_gemm_simt_gated(const void* X, const void* W, void* out, int dtype, int M, int N, int K, int ldx,
                                   int ldo, int epi, int batch, long long sx, long long sw, long long so, int act, float limit,
                                   cudaStream_t stream) {
-    TB_REQUIRE(act >= 0 && act < TB_ACT_KINDS, "gemm: unknown gate %d", act);
+    TB_REQUIRE(act >= 0 && act < (epi == TB_EPI_STORE ? TB_UNARY_KINDS : TB_ACT_KINDS), "gemm: unknown gate or activation %d", act);
     TB_REQUIRE(M > 0 && N > 0 && K > 0, "gemm: sizes must be positive (M=%d N=%d K=%d)", M, N, K);
     TB_REQUIRE(batch > 0 && batch <= 65535, "gemm: a batch of %d products", batch);
     TB_REQUIRE(ldx >= K, "gemm: row stride %d of X is shorter than K=%d", ldx, K);
@@ -178,8 +178,8 @@ extern "C" int tb_gemm_simt_gated(const void* X, const void* W, void* out, int d
     TB_REQUIRE((M + BM - 1) / BM <= 65535, "gemm: M=%d is too large for one launch", M);
     if (epi == TB_EPI_STORE && M <= 16 && batch > 1 && (N + 7) / 8 <= 65535) {      // a decode step's rows: a warp per output
         int r;
-        if (dtype == TB_F32) r = launch_rows<float>(X, W, out, M, N, K, ldx, ldo, epi, batch, sx, sw, so, stream);
-        else if (dtype == TB_BF16) r = launch_rows<__nv_bfloat16>(X, W, out, M, N, K, ldx, ldo, epi, batch, sx, sw, so, stream);
+        if (dtype == TB_F32) r = launch_rows<float>(X, W, out, M, N, K, ldx, ldo, epi, batch, sx, sw, so, act, stream);
+        else if (dtype == TB_BF16) r = launch_rows<__nv_bfloat16>(X, W, out, M, N, K, ldx, ldo, epi, batch, sx, sw, so, act, stream);
         else { tb_set_error("gemm: unknown dtype %d", dtype); return 1; }
         if (r) return r;
         TB_CHECK_LAUNCH("gemm_rows");
@@ -204,15 +204,17 @@ extern "C" int tb_gemm_simt(const void* X, const void* W, void* out, int dtype, 
     return tb_gemm_simt_batched(X, W, out, dtype, M, N, K, ldx, ldo, epi, 1, 0, 0, 0, stream);
 }
 
+// ``act``: the activation of the STORE epilogue (activation.h).
 // out (epilogue store, float32 or add) = X[M,K] . W[N,K]^T for a few rows and a small matrix, a warp per output element:
 // the products of a decode step whose matrices are too small to pay for a tensor-core launch (a router, a narrow gate).
 extern "C" int tb_gemm_rows(const void* X, const void* W, void* out, int dtype, int M, int N, int K, int ldx, int ldo, int epi,
-                            cudaStream_t stream) {
+                            int act, cudaStream_t stream) {
+    TB_REQUIRE(epi == TB_EPI_STORE ? act >= 0 && act < TB_UNARY_KINDS : act == 0, "gemm_rows: unknown activation %d", act);
     TB_REQUIRE(M > 0 && N > 0 && K > 0 && M <= 65535 && (N + 7) / 8 <= 2147483647, "gemm_rows: sizes (M=%d N=%d K=%d)", M, N, K);
     TB_REQUIRE(ldx >= K, "gemm_rows: row stride %d of X is shorter than K=%d", ldx, K);
     int r;
-    if (dtype == TB_F32) r = launch_rows<float>(X, W, out, M, N, K, ldx, ldo, epi, 1, 0, 0, 0, stream);
-    else if (dtype == TB_BF16) r = launch_rows<__nv_bfloat16>(X, W, out, M, N, K, ldx, ldo, epi, 1, 0, 0, 0, stream);
+    if (dtype == TB_F32) r = launch_rows<float>(X, W, out, M, N, K, ldx, ldo, epi, 1, 0, 0, 0, act, stream);
+    else if (dtype == TB_BF16) r = launch_rows<__nv_bfloat16>(X, W, out, M, N, K, ldx, ldo, epi, 1, 0, 0, 0, act, stream);
     else { tb_set_error("gemm_rows: unknown dtype %d", dtype); return 1; }
     if (r) return r;
     TB_CHECK_LAUNCH("gemm_rows");

@@ -101,7 +101,7 @@ struct TcArgs {
     // 1/sqrt(mean(x^2) + eps) in its epilogue, or (K cut into slices: no CTA sees a whole row) leaves its rows'
     // partial sums of squares at sumsq_out [slice][32] for the consumer of the sums to add up, in slice order, and apply
     const float* xf; int ldxf; const float* norm_w; float* sumsq_out; float norm_eps;
-    int act; float limit;   // the gate of the SWIGLU epilogue (activation.h); 0: silu
+    int act; float limit;   // the gate of the SWIGLU epilogue (0: silu), or the activation of the STORE epilogue (0: none) (activation.h)
 };
 
 // TMA ring depth.  Decode tiles (BN <= 64) take as many stages as still let two CTAs share an SM: the
@@ -122,7 +122,11 @@ template <int BN, bool SWAP, int STAGES = stages_for<BN>()> constexpr size_t sme
 
 // Plain mode: the epilogue of one 32-column chunk held by one thread (row = token m, columns = outputs col0 + j).
 template <int EPI, int NV>
-__device__ __forceinline__ void epilogue_chunk(const float* v, const TcArgs& a, int row, int col0, int lane) {
+__device__ __forceinline__ void epilogue_chunk(float* v, const TcArgs& a, int row, int col0, int lane) {
+    if (EPI == TB_EPI_STORE && a.act != TB_UNARY_NONE) {
+#pragma unroll
+        for (int j = 0; j < NV; ++j) v[j] = tb_unary(a.act, v[j]);
+    }
     {
         const int m = row;
         if (m >= a.rows_a) return;
@@ -234,7 +238,7 @@ __device__ __forceinline__ void epilogue_rows(const float* val, float* tile, con
             if (row0 + r >= a.rows_a) continue;
             const float v = tile[r * 33 + lane];
             if (EPI == TB_EPI_F32) o[(size_t)r * a.ldo] = v;
-            else ((__nv_bfloat16*)a.out)[(size_t)(row0 + r) * a.ldo + col] = __float2bfloat16_rn(v);
+            else ((__nv_bfloat16*)a.out)[(size_t)(row0 + r) * a.ldo + col] = __float2bfloat16_rn(tb_unary(a.act, v));
         }
     }
 }
@@ -267,7 +271,10 @@ __device__ __forceinline__ void swap_tile_out(const float* part, const TcArgs& a
         for (int item = t; item < BN * 32; item += 128) {
             const int m = item >> 5, n0 = tile_a * BM + (item & 31) * 4;
             if (m >= a.rows_b || n0 >= a.rows_a) continue;
-            const float4 f = *reinterpret_cast<const float4*>(part + m * BM + (item & 31) * 4);
+            float4 f = *reinterpret_cast<const float4*>(part + m * BM + (item & 31) * 4);
+            if (EPI == TB_EPI_STORE && a.act != TB_UNARY_NONE) {
+                f.x = tb_unary(a.act, f.x); f.y = tb_unary(a.act, f.y); f.z = tb_unary(a.act, f.z); f.w = tb_unary(a.act, f.w);
+            }
             const bool whole = n0 + 4 <= a.rows_a;
             if (EPI == TB_EPI_STORE) {
                 __nv_bfloat16* o = (__nv_bfloat16*)a.out + (size_t)m * a.ldo + n0;
@@ -1141,11 +1148,11 @@ extern "C" int tb_gemm_tc_normed(const float* xf, int ldxf, const float* norm_w,
 // splits: K slices (swap mode, ADD epilogue only); 0 = choose; -1 = choose, and add the parts of a sum in a fixed order
 // (swap mode: the slices of a tile form a thread-block cluster; prompt products: no tile is cut along K), so that
 // the same inputs give the same bits on every run.
-// act, limit: the gate of the SWIGLU epilogue (activation.h).
+// act, limit: the gate of the SWIGLU epilogue, or the activation of the STORE epilogue (activation.h).
 extern "C" int tb_gemm_tc_gated(const void* X, const void* W, void* out, int M, int N, int K, int ldx, int ldo, int epi,
                                 int splits, int act, float limit, cudaStream_t stream) {
     if (tb_gemm_tc_check(M, N, K, ldx, ldo, epi, X, W, out)) return 1;
-    TB_REQUIRE(act >= 0 && act < TB_ACT_KINDS, "gemm_tc: unknown gate %d", act);
+    TB_REQUIRE(act >= 0 && act < (epi == TB_EPI_STORE ? TB_UNARY_KINDS : TB_ACT_KINDS), "gemm_tc: unknown gate or activation %d", act);
     const bool ordered = splits < 0;
     if (ordered) splits = 0;
     const bool swap = M < g_swap_below;

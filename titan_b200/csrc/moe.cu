@@ -2,7 +2,8 @@
 //
 //   tb_moe_route     one warp a token: the ``top`` largest of its E router logits (float32; the lowest index wins a
 //                    tie), their weights = softmax over the chosen logits only, and, if the router's row has one more
-//                    column, the sigmoid of that column (the gate of an expert that every token uses).
+//                    column, the sigmoid of that column (the gate of an expert that every token uses).  A bias (one
+//                    number an expert) joins the logits first, for the choice and the weights alike.
 //                    Token t's k-th choice is *pair* t * top + k.
 //   tb_moe_plan      one block: pairs grouped by expert (``perm``: sorted place -> pair), and the list of row tiles
 //                    (expert, first sorted row, rows) that the grouped product's blocks work through.
@@ -65,7 +66,7 @@ __device__ __forceinline__ void route_row(float* mine, int E, int top, int has_g
     if (has_gate && lane == 0) gate[t] = 1.0f / (1.0f + expf(-gate_logit));
 }
 
-__global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ z, int ldz, int E, int top, int has_gate,
+__global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict__ z, int ldz, const float* __restrict__ bias, int E, int top, int has_gate,
                                                         int* __restrict__ ids, float* __restrict__ wts, float* __restrict__ gate, int T_) {
     pdl_launch_dependents();
     pdl_wait();
@@ -75,7 +76,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float* __restrict_
     if (t >= T_) return;
     float* mine = sm + (size_t)warp * E;
     const float* row = z + (size_t)t * ldz;
-    for (int e = lane; e < E; e += 32) mine[e] = row[e];
+    for (int e = lane; e < E; e += 32) mine[e] = row[e] + (bias ? bias[e] : 0.f);
     __syncwarp();
     route_row(mine, E, top, has_gate, has_gate ? row[E] : 0.f, ids, wts, gate, t, lane);
 }
@@ -397,12 +398,12 @@ __global__ void moe_combine_kernel(const float* __restrict__ y, const float* __r
 
 }  // namespace
 
-extern "C" int tb_moe_route(const float* z, int ldz, int E, int top, int has_gate, int* ids, float* wts, float* gate,
+extern "C" int tb_moe_route(const float* z, int ldz, const float* bias, int E, int top, int has_gate, int* ids, float* wts, float* gate,
                             int T_, cudaStream_t stream) {
     TB_REQUIRE(T_ > 0 && E > 0 && top > 0 && top <= E, "moe_route: %d of %d experts", top, E);
     TB_REQUIRE(E <= 2048, "moe_route: %d experts (at most 2048)", E);
     TB_REQUIRE(ldz >= E + (has_gate ? 1 : 0) && z && ids && wts && (!has_gate || gate), "moe_route: missing buffers");
-    tb_launch(moe_route_kernel, (T_ + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream, z, ldz, E, top, has_gate, ids, wts, gate, T_);
+    tb_launch(moe_route_kernel, (T_ + 3) / 4, 128, (size_t)4 * E * sizeof(float), stream, z, ldz, bias, E, top, has_gate, ids, wts, gate, T_);
     TB_CHECK_LAUNCH("moe_route");
     return 0;
 }

@@ -1,8 +1,9 @@
 """A decoder assembled from a ``ModelSpec``: embedding, blocks in their running order,
 final norm and LM head.
 
-The running order is data (``ModelSpec.order``): it may name a layer twice, and
-a layer's mixer may read another layer's cache (``MixerSpec.cache_from``).
+The running order is data (``ModelSpec.order``): it may name a layer twice (with
+``ModelSpec.loop``, whole stretches of layers run in passes, each entered through
+``parts.loop.LoopEntry``), and a layer's mixer may read another layer's cache (``MixerSpec.cache_from``).
 berniehans/titan hard-codes ``for layer in 0..L`` (engine/engine-core/src/
 forward_driver.rs:988, 2149-2334) and computes logits for the last position
 only (:1215-1238); here the wanted rows are gathered before the final norm, so
@@ -17,6 +18,7 @@ import torch
 from .. import kernels as K
 from ..cache.groups import CacheNeed
 from ..parts import NORMS, build_block, declare_weights, linear
+from ..parts.loop import LoopEntry
 from ..weights.loader import WeightSource, WeightSpec
 
 
@@ -27,6 +29,7 @@ class DecoderModel:
         self.blocks = [build_block(layer) for layer in spec.layers]
         self.final_norm = NORMS.build(spec.final_norm)
         self.embedding_norm = None if spec.embedding_norm is None else NORMS.build(spec.embedding_norm)
+        self.loop = None if spec.loop is None else LoopEntry(spec.loop, spec.hidden_size)
         self.embedding: Optional[torch.Tensor] = None
         self.shared = {}
         self.lm_head: Optional[torch.Tensor] = None
@@ -55,6 +58,8 @@ class DecoderModel:
             b.bind(get)
             if hasattr(b, "bind_shared"):
                 b.bind_shared(self.shared)
+        if self.loop is not None:
+            self.loop.bind(get)
         self.final_norm.bind(get)
         if self.embedding_norm is not None:
             self.embedding_norm.bind(get)
@@ -73,6 +78,9 @@ class DecoderModel:
                 for v in vars(part).values():
                     if isinstance(v, torch.Tensor):
                         add(v)
+        if self.loop is not None:
+            for t in (self.loop.w_x, self.loop.w_x0, self.loop.step):
+                add(t)
         add(self.lm_head)
         add(self.final_norm.weight)
         return total
@@ -94,9 +102,15 @@ class DecoderModel:
             ctx.scratch["row_sums"] = torch.zeros((len(self.spec.order), 16, 32), dtype=torch.float32, device=ctx.device)
         ctx.runs = runs = len(self.spec.order)
         ctx.block_state = lambda run: cache.view_for_layer(runs + run)      # (holds no reference to ctx: a cycle would keep the step's tensors until the collector runs)
+        if self.loop is not None:
+            self.loop.begin(x, ctx)
         for run, i in enumerate(self.spec.order):
             ctx.run = run
+            if self.loop is not None and self.loop.spec.pass_at(run) is not None:
+                self.loop.enter(x, ctx, self.loop.spec.pass_at(run))
             ctx.next_block = self.blocks[self.spec.order[run + 1]] if run + 1 < len(self.spec.order) else None
+            if self.loop is not None and self.loop.spec.pass_at(run + 1) is not None:
+                ctx.next_block = self.loop         # the residual rows change again before the next block reads them
             self.blocks[i].forward(x, ctx, cache.view_for_layer(self.cache_run_of(run)))
             if ctx.after_layer is not None:    # an observer of the residual stream after every run of a layer (tests, debugging)
                 ctx.after_layer(run, self._stream_sum(x, ctx, peek=True))

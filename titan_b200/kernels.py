@@ -21,6 +21,9 @@ F32, BF16 = 0, 1
 # What the SWIGLU epilogue makes of a (gate, up) pair of sums (csrc/activation.h): silu(g) u; gelu_tanh(g) u; or, with
 # g' = min(g, limit) and u' = clamp(u, -limit, limit), g' sigmoid(1.702 g') (u' + 1).
 ACT_SILU, ACT_GELU_TANH, ACT_SWISH_CLAMPED = 0, 1, 2
+# Activations of one sum, for the STORE epilogue: none, or max(z, 0)^2
+UNARY_NONE, UNARY_RELU2 = 0, 1
+UNARIES = {"relu2": UNARY_RELU2}
 GATES = {"silu": ACT_SILU, "gelu_tanh": ACT_GELU_TANH, "swish_clamped": ACT_SWISH_CLAMPED}
 
 launch_count = 0          # launcher calls since import (a launcher starts one or two kernels)
@@ -155,6 +158,16 @@ class ShiftNormArgs(Structure):
                 ("rows_per_block", c_int)]
 
 
+class ConvQkvArgs(Structure):
+    """Arguments of the kernel between a fused Q | K | V projection and its attention where the projected channels pass a short
+    causal convolution over time (csrc/conv_qkv.cu)."""
+    _fields_ = [("inp", c_void_p), ("in_stride", c_int), ("taps", c_void_p), ("n_taps", c_int), ("state", c_void_p), ("state_stride", c_longlong),
+                ("q_out", c_void_p), ("q_stride", c_int), ("kv_out", c_void_p), ("kv_stride", c_int), ("rope", RotaryArgs),
+                ("nh", c_int), ("nkv", c_int), ("hd", c_int),
+                ("q_start", c_void_p), ("start_pos", c_void_p), ("kv_len", c_void_p), ("slot_of_seq", c_void_p),
+                ("cache", KvView), ("append", c_int), ("zero_in", c_int), ("T", c_int), ("B", c_int), ("max_new", c_int)]
+
+
 class WkvArgs(Structure):
     """Arguments of the wkv mixer's kernels (csrc/wkv.cu)."""
     _fields_ = [("h", c_void_p), ("h_stride", c_int), ("mixes", c_void_p), ("mix_stride", c_int), ("mu", c_void_p),
@@ -243,7 +256,9 @@ def lib():
         l.tb_rotary_rows.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_int, POINTER(RotaryArgs), c_int, c_float, c_void_p]
         l.tb_gemm_simt_batched.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                                            c_longlong, c_longlong, c_longlong, c_void_p]
-        l.tb_gemm_rows.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
+        l.tb_gemm_rows.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
+        l.tb_conv_qkv.argtypes = [POINTER(ConvQkvArgs), c_int, c_int, c_int, c_void_p]
+        l.tb_pass_entry.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p]
         l.tb_rmsnorm_add.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_void_p]
         l.tb_round_rows.argtypes = [c_void_p, c_void_p, c_longlong, c_void_p]
         l.tb_gelu_mul_table.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
@@ -251,7 +266,7 @@ def lib():
         l.tb_latent_append.argtypes = [c_void_p, c_int, c_int, POINTER(KvView), POINTER(Batch), c_void_p]
         l.tb_lightning_scan.argtypes = [POINTER(LightningArgs), c_int, c_void_p]
         l.tb_gated_rmsnorm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p]
-        l.tb_moe_route.argtypes = [c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
+        l.tb_moe_route.argtypes = [c_void_p, c_int, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_int, c_void_p]
         l.tb_token_gate_rows.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
         l.tb_moe_plan_tiles.argtypes = [c_int, c_int]
         l.tb_moe_plan.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p, c_void_p, c_void_p]
@@ -388,7 +403,7 @@ def rmsnorm(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor, eps: float, strea
 
 def gemm_simt(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: int, stream: int, gate: int = ACT_SILU, limit: float = 0.0) -> None:
     """out (epilogue ``epi``) = x[M,K] . w[N,K]^T; x and out may be row-strided views.  ``gate``, ``limit``: what the
-    SWIGLU epilogue makes of a pair (ACT_*)."""
+    SWIGLU epilogue makes of a pair (ACT_*), or the STORE epilogue of a sum (``gate`` = UNARY_*)."""
     _need_cuda(x, w, out)
     M, K = x.shape
     N = w.shape[0]
@@ -412,9 +427,9 @@ def gemm_simt_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: 
                                       out.stride(0), epi, batch, x_step, N * K, out_step, stream))
 
 
-def gemm_rows(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: int, stream: int) -> None:
+def gemm_rows(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: int, stream: int, unary: int = UNARY_NONE) -> None:
     """out (epilogue store, float32 or add) = x[M,K] . w[N,K]^T, a warp per output element: for the few rows of a decode step and
-    matrices too small to pay for a tensor-core launch."""
+    matrices too small to pay for a tensor-core launch.  ``unary``: the STORE epilogue's activation (UNARY_*)."""
     _need_cuda(x, w, out)
     M, K = x.shape
     if w.shape[1] != K or not w.is_contiguous() or x.stride(1) != 1 or out.stride(1) != 1 or x.dtype != w.dtype:
@@ -422,7 +437,7 @@ def gemm_rows(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epi: int, str
     want = w.dtype if epi == EPI_STORE else torch.float32
     if out.dtype != want:
         raise KernelError(f"gemm_rows: this epilogue writes {want}, the output is {out.dtype}")
-    _check(lib().tb_gemm_rows(x.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(w.dtype), M, w.shape[0], K, x.stride(0), out.stride(0), epi, stream))
+    _check(lib().tb_gemm_rows(x.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(w.dtype), M, w.shape[0], K, x.stride(0), out.stride(0), epi, int(unary), stream))
 
 
 def rmsnorm_add(y: torch.Tensor, w: torch.Tensor, x: torch.Tensor, eps: float, stream: int,
@@ -629,6 +644,21 @@ def qkv_whole_norm(args: "WholeNormArgs", out_dtype: torch.dtype, stream: int) -
     _check(lib().tb_qkv_whole_norm(byref(args), dtype_code(out_dtype), stream))
 
 
+def conv_qkv(args: "ConvQkvArgs", in_dtype: torch.dtype, out_dtype: torch.dtype, stream: int, any_size: bool = False) -> None:
+    _check(lib().tb_conv_qkv(byref(args), dtype_code(in_dtype), dtype_code(out_dtype), int(any_size), stream))
+
+
+def pass_entry(x: torch.Tensor, base: Optional[torch.Tensor], step: Optional[torch.Tensor], lowp: Optional[torch.Tensor], stream: int) -> None:
+    """lowp = x in its dtype; x <- base + step (float32 rows; ``base`` None: x itself, ``step`` a vector or None: zeros)."""
+    _need_cuda(x, base, step, lowp)
+    if x.dtype != torch.float32 or any(t is not None and (t.dtype != torch.float32 or not t.is_contiguous()) for t in (x, base, step)) \
+            or (base is not None and base.shape != x.shape) or (step is not None and step.numel() != x.shape[1]) \
+            or (lowp is not None and (lowp.shape != x.shape or not lowp.is_contiguous())):
+        raise KernelError("pass_entry: contiguous float32 rows of one shape and a vector as wide as they are wanted")
+    _check(lib().tb_pass_entry(x.data_ptr(), _ptr(base), _ptr(step), _ptr(lowp), dtype_code(lowp.dtype) if lowp is not None else F32, x.shape[0],
+                               x.shape[1], stream))
+
+
 def attn_mixed_prefill(args: AttnArgs, dtype: torch.dtype, stream: int) -> None:
     _check(lib().tb_attn_mixed_prefill(byref(args), dtype_code(dtype), stream))
 
@@ -691,11 +721,13 @@ def gated_rmsnorm(o: torch.Tensor, w: torch.Tensor, gate: torch.Tensor, y: torch
 
 
 def moe_route(z: torch.Tensor, experts: int, top: int, has_gate: bool, ids: torch.Tensor, wts: torch.Tensor,
-              gate: Optional[torch.Tensor], stream: int) -> None:
+              gate: Optional[torch.Tensor], stream: int, bias: Optional[torch.Tensor] = None) -> None:
     """Per row of z (float32 [T, experts (+1)]): the ``top`` largest logits' indices and their softmax weights; the last
-    column's sigmoid into ``gate`` if the row has one more column than experts."""
-    _need_cuda(z, ids, wts, gate)
-    _check(lib().tb_moe_route(z.data_ptr(), z.stride(0), experts, top, int(has_gate), ids.data_ptr(), wts.data_ptr(), _ptr(gate),
+    column's sigmoid into ``gate`` if the row has one more column than experts.  ``bias`` (float32 [experts]) joins the logits first."""
+    _need_cuda(z, ids, wts, gate, bias)
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != experts or not bias.is_contiguous()):
+        raise KernelError(f"moe_route: a float32 bias of {experts} numbers is wanted")
+    _check(lib().tb_moe_route(z.data_ptr(), z.stride(0), _ptr(bias), experts, top, int(has_gate), ids.data_ptr(), wts.data_ptr(), _ptr(gate),
                               z.shape[0], stream))
 
 

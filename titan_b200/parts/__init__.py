@@ -6,7 +6,7 @@ from typing import List
 from ..weights.loader import WeightSpec
 from .base import (BLOCKS, FEED_FORWARDS, MIXERS, NORMS, POSITIONS, FeedForward, Mixer, Norm, Part,
                    PositionEncoding, Registry)
-from . import attention, block, diff_attention, gated_delta, latent_attention, lightning, mlp, mlstm, moe, norm, parallel, retention, rotary, token_table, wkv  # noqa: F401  (registration)
+from . import attention, block, diff_attention, gated_delta, latent_attention, lightning, loop, mlp, mlstm, moe, norm, parallel, retention, rotary, token_table, wkv  # noqa: F401  (registration)
 
 
 def build_block(layer_spec):
@@ -20,6 +20,8 @@ def declare_weights(model_spec) -> List[WeightSpec]:
     """Every tensor the model owns, in file order, without touching a device."""
     specs = [WeightSpec(model_spec.embedding, (model_spec.vocab_size, model_spec.hidden_size))]
     specs += [WeightSpec(name, tuple(shape)) for name, shape in model_spec.shared_tensors]
+    if model_spec.loop is not None:
+        specs += loop.LoopEntry(model_spec.loop, model_spec.hidden_size).weight_specs()
     for layer in model_spec.layers:
         specs += build_block(layer).weight_specs()
     if model_spec.embedding_norm is not None:

@@ -50,6 +50,13 @@ Options of the spec (``MixerSpec.extra``) beyond the common fields:
   ``head_mix`` = name of a [heads, heads] tensor M: head h's score becomes sum_g M[h, g] * score_g, for every (query, key) pair,
   before the softmax.
   ``head_gate`` = name of a [heads, hidden] tensor: head h's output is multiplied by sigmoid(W h)_h, one number a head.
+* ``sink_value``: a number that every head's denominator takes as a sink, where it is a constant of the design (0: softmax with one
+  added below the line).
+* ``exact_weights``: softmax weights meet the values with sixteen bits instead of eight in the tensor-core kernels.
+* ``conv`` = n: each channel of q, k and v passes a causal convolution of n taps over time straight behind its projection, before the
+  rotation: tensors ``<name>.conv`` [channels, n], the last tap on the current token, zeros before the sequence's start
+  (``csrc/conv_qkv.cu``).  The last n - 1 projected rows of a sequence are a float32 row of a ``state`` cache group beside the keys and
+  values.  No head norm and no normed or blended values beside it.
 * ``value_mix`` = (first, name): values are blended across layers.  ``first`` None: this layer's values are what the
   others blend with, and it keeps them for the step; else v <- (1 - l) v + l v_first with l the tensor ``name`` and
   v_first the values of layer ``first`` for the same tokens.  The blended values are what the cache holds.
@@ -63,7 +70,7 @@ from typing import List, Optional
 import torch
 
 from .. import kernels as K
-from ..cache.groups import CacheNeed, KVGroup
+from ..cache.groups import CacheNeed, KVGroup, StateGroup
 from ..weights.loader import WeightSpec
 from . import linear
 from .base import MIXERS, POSITIONS, Mixer
@@ -178,6 +185,17 @@ class AttentionMixer(Mixer):
                 _, rows, far = self.rel_spec
                 if rows < 1 or (rows >= 2 and not far > rows // 2):
                     raise ValueError(f"a distance table of {rows} rows that reaches its last row at distance {far}")
+        self.exact_weights = bool(s.option("exact_weights", False))
+        self.sink_value = s.option("sink_value")
+        if self.sink_value is not None and (self.sink_name or self.shaped):
+            raise ValueError("a constant sink takes the place of a learned one, and comes without shaped scores")
+        self.taps, self.conv_w = s.option("conv"), None
+        if self.taps is not None:
+            self.folds_norm, self.extended, self.taps = False, True, int(self.taps)
+            if not 1 <= self.taps <= 64:
+                raise ValueError(f"a convolution of {self.taps} taps (1 to 64)")
+            if self.shaped or self.shared or self.unit_norm or self.value_mix is not None or self.value_norm is not None or s.qk_norm is not None:
+                raise ValueError("a convolution on q, k and v comes without head norms, normed or blended values, shaped scores or another layer's cache")
         self.bias = self.b_o = self.whole_q_w = self.whole_k_w = self.rel_table = self.head_mix = None
 
     # -- declaration ------------------------------------------------------ #
@@ -185,7 +203,10 @@ class AttentionMixer(Mixer):
         if self.shared:
             return None
         # kept first tokens stay in reach for good: such a window is a mask over a cache that keeps every key, not a ring
-        return CacheNeed("kv", self.spec.num_kv_heads, self.hd, None if self.keep_first else self.spec.window)
+        kv = CacheNeed("kv", self.spec.num_kv_heads, self.hd, None if self.keep_first else self.spec.window)
+        if self.taps is None or self.taps == 1:
+            return kv
+        return kv, CacheNeed("state", state_shape=((self.taps - 1) * (self.Q + 2 * self.KV),), state_dtype=torch.float32)
 
     def _names(self):
         """Tensor names (relative to the prefix) by role; "qkv" only if the spec names a fused tensor."""
@@ -209,6 +230,11 @@ class AttentionMixer(Mixer):
             if not self.shared:
                 specs += [WeightSpec(p + n["k"], (s.num_kv_heads * kd, s.hidden_size)),
                           WeightSpec(p + n["v"], (s.num_kv_heads * vd, s.hidden_size))]
+        if self.taps is not None:
+            if n["qkv"] is not None:
+                raise ValueError("the taps of a convolution belong to three separate projections")
+            specs += [WeightSpec(p + n[r] + ".conv", (rows, self.taps), "vector", ("normal_around", 0.3, 0.3))
+                      for r, rows in (("q", s.num_heads * kd), ("k", s.num_kv_heads * kd), ("v", s.num_kv_heads * vd))]
         if self.sink_name:
             specs.append(WeightSpec(p + self.sink_name, (s.num_heads,), "vector", ("normal", 1.0)))
         if self.gate_name:
@@ -250,6 +276,11 @@ class AttentionMixer(Mixer):
             self.w_o = torch.nn.functional.pad(w, (0, self.hd - self.value_dim)).reshape(s.hidden_size, self.Q).contiguous()
         if self.sink_name:
             self.sink = get(p + self.sink_name)
+        if self.sink_value is not None:
+            self.sink = torch.full((s.num_heads,), float(self.sink_value), dtype=torch.float32, device=self.w_o.device)
+        if self.taps is not None:                     # [taps, channels], padded like the projections
+            rows = (("q", s.num_heads, self.key_dim), ("k", s.num_kv_heads, self.key_dim), ("v", s.num_kv_heads, self.value_dim))
+            self.conv_w = torch.cat([self._padded_rows(get(p + n[r] + ".conv").float(), heads, dim) for r, heads, dim in rows]).t().contiguous()
         if self.gate_name:
             self.w_gate = self._padded_rows(get(p + self.gate_name), s.num_heads, self.value_dim)
         if self.value_mix is not None and self.value_mix[0] is not None:
@@ -324,6 +355,29 @@ class AttentionMixer(Mixer):
         qa.kv_len = lay.kv_len.data_ptr()
         return qa
 
+    def _convolve(self, src, width, q_buf, q_stride, kv_rows, view, state, rope, ctx, append: bool, zero_in: bool) -> None:
+        """Convolution over time, rotation and append: the projected rows ``src`` become queries, and keys and values in the cache and
+        (``kv_rows`` = address and stride, or None) beside it."""
+        s, lay = self.spec, ctx.layout
+        a = K.ConvQkvArgs()
+        a.inp, a.in_stride = src.data_ptr(), width
+        a.taps, a.n_taps = self.conv_w.data_ptr(), self.taps
+        if state is not None:
+            group, index = state
+            if not isinstance(group, StateGroup):
+                raise TypeError(f"the convolution keeps its window in a 'state' cache group, not in {type(group).__name__}")
+            rows = group.layer_storage(index)
+            a.state, a.state_stride = rows.data_ptr(), rows.stride(0)
+        a.q_out, a.q_stride = q_buf.data_ptr(), q_stride
+        if kv_rows is not None:
+            a.kv_out, a.kv_stride = kv_rows
+        a.rope, a.nh, a.nkv, a.hd = rope, s.num_heads, s.num_kv_heads, self.hd
+        a.q_start, a.start_pos = lay.q_start.data_ptr(), lay.start_pos.data_ptr()
+        a.kv_len, a.slot_of_seq = lay.kv_len.data_ptr(), lay.slot_of_seq.data_ptr()
+        a.cache, a.append, a.zero_in = view, int(append), int(zero_in)
+        a.T, a.B, a.max_new = lay.T, lay.B, lay.max_new
+        K.conv_qkv(a, src.dtype, q_buf.dtype, ctx.stream, any_size=not ctx.options.get("conv_vectors", True))
+
     def _forward_shaped(self, h, ctx, cache, out: torch.Tensor) -> None:
         """Biases, norms over the whole projection, shaped and blended scores, one gate a head: one float32 product
         (Q | K | V | gate logits), the kernel that adds biases, norms, rounds and appends, the mixed-heads attention, the
@@ -391,6 +445,9 @@ class AttentionMixer(Mixer):
         s, lay = self.spec, ctx.layout
         T, Q, KV, hd = lay.T, self.Q, self.KV, self.hd
         width = Q if self.shared else Q + 2 * KV
+        window_state = None
+        if self.taps is not None and self.taps > 1:
+            cache, window_state = cache
         view = self._view(cache)
         decode = lay.all_single
         rope = self.position.kernel_args(ctx.device)
@@ -424,6 +481,12 @@ class AttentionMixer(Mixer):
         # they replace: always for single tokens and for caches that keep everything; in a ring only if
         # every sequence starts at position 0 (attention then reads the step's own rows alone).
         append_now = not self.shared and (decode or view.ring_rows == 0 or lay.all_fresh)
+        if self.taps is not None:
+            projected = qkv
+            if not wide_sum:                                   # later tokens of a run read the projected rows: the results go elsewhere
+                qkv = q_buf = ctx.empty((T, width))
+            beside = None if decode else (qkv.data_ptr() + Q * qkv.element_size(), width)
+            self._convolve(projected, width, q_buf, q_stride, beside, view, window_state, rope, ctx, append=append_now, zero_in=wide_sum)
         qa = self._qk_args(qkv, width, q_buf, q_stride, view, lay, rope, T, hd, append=append_now, zero_in=wide_sum)
         if not (self.shared or wide_sum):
             qa.k_out, qa.k_stride = qkv.data_ptr() + Q * qkv.element_size(), width
@@ -453,7 +516,7 @@ class AttentionMixer(Mixer):
             # the normed values are what a prompt's attention reads: written back over the step's own V columns
             qa.v_keep, qa.v_keep_stride = qkv.data_ptr() + (Q + KV) * qkv.element_size(), width
         folds_head_norm = wide_sum and ctx.options.get("fold_head_norm", True) and not self.extended
-        if not folds_head_norm:
+        if not folds_head_norm and self.taps is None:
             K.qk_norm_rope(qa, qkv.dtype, q_buf.dtype, ctx.stream)
 
         attn = ctx.empty((T, Q))
@@ -465,6 +528,7 @@ class AttentionMixer(Mixer):
         aa.window, aa.scale = s.window or 0, self.scale
         aa.sink = None if self.sink is None else self.sink.data_ptr()
         aa.keep_first = self.keep_first if s.window else 0
+        aa.exact_weights = int(self.exact_weights)
         if decode:
             fast = ctx.options.get("attention", "fast") != "plain" and q_buf.dtype == torch.bfloat16 and hd in (64, 128)
             chunk, splits = decode_split(lay, view.kv_heads, ctx.options, fast)

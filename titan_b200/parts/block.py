@@ -385,7 +385,8 @@ class SandwichBlock(Part):
         x <- sum over j = 0 .. i + 1 of w_j X_j             X_0 the rows that entered the first block, X_{j+1} what block j made
 
     ``LayerSpec.norms`` are the norms after the sublayers (one a sublayer; the feed-forward, with both its norms, may be
-    absent).  ``LayerSpec.extra``: "token_shift" = name of the factors s [W]; "depth_average" = (name of the weights w [i + 2], i)
+    absent).  ``LayerSpec.extra``: "scales" = names of vectors [W], one a sublayer, that its normed result is multiplied by before it
+    is added ("layer scale"; the vector and the norm's weight are one factor, formed once, in float32); "token_shift" = name of the factors s [W]; "depth_average" = (name of the weights w [i + 2], i)
     with i the block's place in the running order.
 
     A sublayer adds into a zeroed float32 buffer of the step; ONE kernel then norms that buffer, adds it to the residual stream,
@@ -397,6 +398,9 @@ class SandwichBlock(Part):
     The rows X_j live in one scratch buffer ([runs, T, W] float32); none of them outlasts its step."""
 
     def __init__(self, spec):
+        names = tuple(spec.option("scales", ()))
+        if names and len(names) != len(spec.norms):
+            raise ValueError(f"{len(names)} scale vectors with {len(spec.norms)} norms after sublayers")
         if spec.mixer_norm is None or (spec.feed_forward is None) != (spec.feed_forward_norm is None) or len(spec.norms) != (1 if spec.feed_forward is None else 2):
             raise ValueError("the sandwich arrangement takes a norm before and a norm after the mixer, and a feed-forward with two norms of its own or none")
         for n in (spec.mixer_norm, spec.feed_forward_norm) + tuple(spec.norms):
@@ -412,6 +416,7 @@ class SandwichBlock(Part):
         self.shift_name = spec.option("token_shift")
         self.depth_name, self.place = spec.option("depth_average", (None, 0))
         self.shift = self.depth_w = None
+        self.scale_names, self.after_w = names, []
 
     def parts(self):
         ffn = () if self.feed_forward is None else (self.feed_forward_norm, self.feed_forward)
@@ -424,6 +429,7 @@ class SandwichBlock(Part):
         out: List[WeightSpec] = []
         for part in self.parts():
             out += part.weight_specs(self.spec.prefix)
+        out += [WeightSpec(self.spec.prefix + n, (self.W,), "vector", ("one_plus_normal", 0.1)) for n in self.scale_names]
         if self.shift_name is not None:
             out.append(WeightSpec(self.spec.prefix + self.shift_name, (self.W,), "vector", ("normal_around", 0.2, 0.3)))
         if self.depth_name is not None:
@@ -434,6 +440,9 @@ class SandwichBlock(Part):
     def bind(self, get) -> None:
         for part in self.parts():
             part.bind(lambda name: get(self.spec.prefix + name))
+        self.after_w = [n.weight for n in self.after]
+        if self.scale_names:
+            self.after_w = [(w.float() * get(self.spec.prefix + n).float()).contiguous() for w, n in zip(self.after_w, self.scale_names)]
         if self.shift_name is not None:
             self.shift = get(self.spec.prefix + self.shift_name).contiguous()
         if self.depth_name is not None:
@@ -489,11 +498,11 @@ class SandwichBlock(Part):
         if self.feed_forward is not None:
             n1, n2 = self.after[0], self.feed_forward_norm
             h = ctx.empty(tuple(x.shape))
-            K.sandwich_join(y, n1.weight, n1.spec.eps, x, ctx.stream, keep=keep, pre_w=n2.weight, pre_eps=n2.spec.eps, h=h)
+            K.sandwich_join(y, self.after_w[0], n1.spec.eps, x, ctx.stream, keep=keep, pre_w=n2.weight, pre_eps=n2.spec.eps, h=h)
             keep = None
             self.feed_forward.forward(h, ctx, y)
         made, n = self._following(x, ctx), self.after[-1]
-        K.sandwich_join(y, n.weight, n.spec.eps, x, ctx.stream, keep=keep, history=history, depth=self.place + 1 if history is not None else 0,
+        K.sandwich_join(y, self.after_w[-1], n.spec.eps, x, ctx.stream, keep=keep, history=history, depth=self.place + 1 if history is not None else 0,
                         depth_w=self.depth_w, **made)
         if made:
             ctx.carried["normed_rows"] = (made["h"], ctx.run + 1)

@@ -18,6 +18,8 @@ Options of the spec beyond experts, top and the shared expert:
 * ``routing = "sigmoid_all"``: scores s = sigmoid(z), each output on its own; the rest as above, with two more options:
   ``group_best`` = n (a group's score is the sum of its n largest s + correction; 1: its best one) and ``renormalize`` =
   False (the weights are the chosen experts' s as they are).
+* ``router_bias`` = True: a tensor (``router_bias``, by default ``<router>.b``), one number an expert, joins the logits before
+  the choice and the softmax (routing "top_softmax").
 * ``shared_gate`` = False: the shared expert's output is added as it is (no sigmoid gate, no tensor for one).
 * ``identity = n``: the last n router outputs are experts without matrices whose output is the input row itself (times
   the weight); they take part in the scores, the groups and the choice like any other.
@@ -59,6 +61,9 @@ class MixtureOfExperts(FeedForward):
         self.shared_gate = bool(s.option("shared_gate", True))
         if self.group_best < 1 or (not self.scored and (self.group_best != 1 or not self.renormalize)):
             raise ValueError("group_best and renormalize are options of the routings that score all outputs")
+        self.has_bias = bool(s.option("router_bias", False))
+        if self.has_bias and self.scored:
+            raise ValueError("a bias on the router's logits comes with routing 'top_softmax'")
         self.identity = int(s.option("identity", 0))
         self.groups, self.keep = int(s.option("groups", 1)), int(s.option("keep", 1))
         self.E, self.top, self.F = int(s.option("experts", 0)), int(s.option("top", 0)), s.intermediate_size
@@ -72,7 +77,7 @@ class MixtureOfExperts(FeedForward):
             raise ValueError(f"{self.groups} groups over {self.n_all} experts, {self.keep} kept, {self.top} experts a token")
         if self.identity and self.shared_F:
             raise ValueError("a shared expert beside experts without matrices is not supported")
-        self.correction = None
+        self.correction = self.router_bias = None
         self.w_router = self.w_gate_up = self.w_down = self.ws_gate_up = self.ws_down = None
 
     def _names(self):
@@ -82,6 +87,7 @@ class MixtureOfExperts(FeedForward):
         names["shared"] = s.name("shared", "shared.")
         names["shared_gate"] = s.name("shared_gate", "shared.sg")
         names["correction"] = s.name("correction", "correction")
+        names["router_bias"] = s.name("router_bias", names["router"] + ".b")
         return names
 
     def weight_specs(self, prefix: str) -> List[WeightSpec]:
@@ -92,6 +98,8 @@ class MixtureOfExperts(FeedForward):
             q = p + n["expert"].format(e)
             specs += [WeightSpec(q + n["gate"], (self.F, H)), WeightSpec(q + n["up"], (self.F, H)), WeightSpec(q + n["down"], (H, self.F))]
         specs.append(WeightSpec(p + n["router"], (self.n_all, H)))
+        if self.has_bias:
+            specs.append(WeightSpec(p + n["router_bias"], (self.n_all,), "vector", ("normal", 0.5)))
         if self.scored:
             specs.append(WeightSpec(p + n["correction"], (self.n_all,), "vector", ("normal", 0.02)))
         if self.shared_F:
@@ -116,6 +124,8 @@ class MixtureOfExperts(FeedForward):
         router = get(p + n["router"])
         if self.scored:
             self.correction = get(p + n["correction"])
+        if self.has_bias:
+            self.router_bias = get(p + n["router_bias"]).contiguous()
         if self.shared_F:
             q = p + n["shared"]
             self.w_router = torch.cat([router, get(p + n["shared_gate"])], dim=0).contiguous() if self.shared_gate else router
@@ -139,7 +149,7 @@ class MixtureOfExperts(FeedForward):
             K.moe_route_scored(z, top, self.correction, self.groups, self.keep, ids, wts, ctx.stream,
                                sigmoid=self.routing == "sigmoid_all", group_best=self.group_best, renorm=self.renormalize)
         else:
-            K.moe_route(z, E, top, gate is not None, ids, wts, gate, ctx.stream)
+            K.moe_route(z, E, top, gate is not None, ids, wts, gate, ctx.stream, bias=self.router_bias)
         shared_y = None
         if self.shared_F:
             act_s = ctx.empty((T, self.shared_F))

@@ -7,7 +7,9 @@ dimensions turns by it: (k, k + rotary_dim/2) with ``pairing="half"``,
 the mixers' business: grouped-query attention takes "half", latent attention
 either) (berniehans/titan:
 engine/engine-core/src/forward_cpu.rs:226-241; rotary_dim = head_dim,
-forward_driver.rs:608).  The inverse frequencies are computed in float64 on the
+forward_driver.rs:608).  ``scaling`` = (factor, low, high, original) changes a frequency f by its wavelength 2 pi / f:
+below original / high it stays, above original / low it becomes f / factor, between them
+(1 - s) f / factor + s f with s = (original / wavelength - low) / (high - low).  The inverse frequencies are computed in float64 on the
 host and rounded once to float32; the angle and its sine and cosine are float32
 in the kernel.
 
@@ -15,11 +17,20 @@ in the kernel.
 """
 from __future__ import annotations
 
+import math
 from typing import Dict
 
 import torch
 
 from .base import POSITIONS, PositionEncoding
+
+
+def scaled_frequencies(inv: torch.Tensor, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Frequencies (float64) scaled by wavelength; with low = high there is no stretch between the two."""
+    waves = original * inv / (2.0 * math.pi)                 # original / wavelength
+    s = ((waves - low) / (high - low if high != low else 1.0)).clamp(0.0, 1.0)
+    blended = (1.0 - s) * inv / factor + s * inv
+    return torch.where(waves > high, inv, torch.where(waves < low, inv / factor, blended))
 
 
 class Rotary(PositionEncoding):
@@ -45,6 +56,8 @@ class Rotary(PositionEncoding):
             rot = self.spec.rotary_dim
             k = torch.arange(rot // 2, dtype=torch.float64)
             inv = torch.tensor(self.spec.theta, dtype=torch.float64) ** (-2.0 * k / rot)
+            if self.spec.scaling is not None:
+                inv = scaled_frequencies(inv, *self.spec.scaling)
             self._tables = {"inv_freq": inv.to(torch.float32).to(device)}
         return self._tables
 
