@@ -654,6 +654,19 @@ def pipesun_config(width, layers, heads, experts, top, ff, shared_ff, window, vo
     return {"architecture": "Pipesun", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
 
 
+def potupel_config(width, layers, heads, experts, top, ff, shared_ff, window, vocab=32768, dense=False, loop=True):
+    """A Potupel model of the same sizes (without windows, which the design does not have): attention with heads of 128 behind
+    convolutions of four taps, a quarter as many kv heads, half of a head rotated with scaled frequencies; dense feed-forwards (as wide
+    as what a token uses of a mixture) in the first layer, mixtures with a shared expert in the others (``dense``: every layer with the
+    dense one).  The two middle layers run twice (``loop``: without it every layer once, as in the models beside it)."""
+    moe = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    mixer = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "conv": 4, "scale": 128 ** -0.5,
+             "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}}
+    out = [{"type": "attention", "mixer": mixer, "mlp": {"kind": "dense", "ff": top * ff + shared_ff} if i == 0 or dense else moe} for i in range(layers)]
+    d = {"architecture": "Potupel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "layers": out}
+    return dict(d, loop={"start": 1, "stop": layers - 1, "times": 2}) if loop and layers > 2 else d
+
+
 def qwen3_like(width, layers, heads, ffn, vocab=32768):
     """The dense model of equal size: the same width, depth and heads, and a feed-forward as wide as what one token uses
     of the mixture (its chosen experts and the shared one)."""
@@ -671,7 +684,7 @@ def launcher_times(engine, torch, K, entries):
                          "gated_rmsnorm", "moe_route", "token_gate_rows", "moe_plan", "moe_grouped", "moe_rows", "moe_combine", "moe_experts_tc",
                          "dyt", "scale_add", "wkv", "moe_route_all", "hyper", "polynorm", "gate_rows", "head_norm_gate", "delta_prep",
                          "recurrent_scan", "group_rmsnorm", "residual_group_norm", "qkv_whole_norm", "attn_mixed_prefill", "attn_mixed_decode", "attn_decode_latent",
-                         "rotary_rows", "moe_route_scored", "pair_prep", "pair_combine", "sandwich_join", "shift_norm") if hasattr(K, n)]
+                         "rotary_rows", "moe_route_scored", "pair_prep", "pair_combine", "sandwich_join", "shift_norm", "conv_qkv", "pass_entry") if hasattr(K, n)]
     events, originals = [], {n: getattr(K, n) for n in names}
 
     def wrap(name, f):
@@ -702,12 +715,13 @@ def launcher_times(engine, torch, K, entries):
 
 
 def run_design(args):
-    """``--design tefezen | zadinex | vuvosun | desalorn | pipesun``: prompt and decode throughput of that design at sizes that resemble a
+    """``--design tefezen | zadinex | vuvosun | desalorn | pipesun | potupel``: prompt and decode throughput of that design at sizes that resemble a
     served model's layers (random weights), beside the Qwen3 dense model of equal size and beside the closest design (for zadinex:
     Tefezen, windowed attention, a recurrence, mixtures of experts; for vuvosun: Zadinex with dense feed-forwards, attention
     with a sink and a recurrence over a matrix state; for desalorn: Tefezen, latent attention over a window, decayed linear
     attention, mixtures of experts with a shared one; for pipesun: Tefezen too, for its latent attention and the norms on its
-    sublayers' outputs), and where a step's time goes by launcher."""
+    sublayers' outputs; for potupel, with its loop and every layer once: Zadinex, attention with a sink beside mixtures of experts, and
+    Potupel with dense feed-forwards and every layer once, which is the dense model's like), and where a step's time goes by launcher."""
     import torch
 
     from titan_b200 import Engine, StepEntry, kernels as K
@@ -722,9 +736,12 @@ def run_design(args):
     for sz in sizes:
         row = {"size": sz}
         beside = {"tefezen": ("qwen3",), "zadinex": ("tefezen", "qwen3"), "vuvosun": ("zadinex_dense", "qwen3"),
-                  "desalorn": ("tefezen", "qwen3"), "pipesun": ("tefezen", "qwen3")}[args.design]
+                  "desalorn": ("tefezen", "qwen3"), "pipesun": ("tefezen", "qwen3"),
+                  "potupel": ("potupel_once", "potupel_dense", "zadinex", "qwen3")}[args.design]
         for which in (args.design,) + beside:
-            if which == "pipesun":
+            if which.startswith("potupel"):
+                cfg = potupel_config(**sz, dense=which == "potupel_dense", loop=which == "potupel")
+            elif which == "pipesun":
                 cfg = pipesun_config(**sz)
             elif which == "desalorn":
                 cfg = desalorn_config(**sz)
@@ -783,7 +800,7 @@ def main():
     ap.add_argument("--micro", action="store_true", help="time the layer's kernels alone (CUDA events) and exit; text lines, not the JSON line")
     ap.add_argument("--timeline", type=int, default=0, metavar="BATCH", help="when the CTAs of one captured decode step's kernels start, wait and end "
                     "(needs TITAN_B200_NVCC_FLAGS=-DTB_TIMELINE); text lines, not the JSON line")
-    ap.add_argument("--design", default=None, choices=["tefezen", "zadinex", "vuvosun", "desalorn", "pipesun"], help="prompt and decode throughput of another design at a few sizes beside "
+    ap.add_argument("--design", default=None, choices=["tefezen", "zadinex", "vuvosun", "desalorn", "pipesun", "potupel"], help="prompt and decode throughput of another design at a few sizes beside "
                     "the dense model of equal size; one JSON line of its own, the default workload is not run")
     ap.add_argument("--design-size", type=int, default=None, choices=[0, 1], help="with --design: one of its sizes only")
     args = ap.parse_args()

@@ -9,9 +9,9 @@
 // the block with a sequence's first token of the step reads the old state; it also writes the new one, each thread for its
 // own channels after it has read them.  Sums, angles and the rotation are float32.
 //
-//   conv_qkv_vec_kernel   up to four taps, heads of 16, 32, 64, 128 or 256: a thread owns eight neighbouring channels and slides
-//                         its window over the run in registers (a row is read once, plus n - 1 rows of the run before);
-//                         rotation partners are lanes of the same warp.
+//   conv_qkv_vec_kernel   up to four taps, heads of 16, 32, 64, 128 or 256: a thread owns four neighbouring channels (eight in heads of
+//                         256) and slides its window over the run in registers (a row is read once, plus n - 1 rows of the run
+//                         before); rotation partners, in halves, are lanes of the same warp.
 //   conv_qkv_kernel       any size: a warp a head, a token at a time.
 #include "common.cuh"
 #include "qk_args.h"
@@ -32,39 +32,27 @@ struct ConvQkvArgs {
 
 namespace {
 
+constexpr int RUN = 8, RUN_THREADS = 128;     // tokens and threads of a block of the vector kernel
 constexpr int NT = 4;                       // taps of the vector kernel's window (fewer: the window's oldest rows weigh nothing)
 
-template <typename T> struct Raw8;
-template <> struct Raw8<__nv_bfloat16> {
-    uint4 r;
-    __device__ __forceinline__ void load(const __nv_bfloat16* p) { r = *reinterpret_cast<const uint4*>(p); }
-    __device__ __forceinline__ void clear() { r = make_uint4(0u, 0u, 0u, 0u); }
-    __device__ __forceinline__ void get(float* o) const {
-        const uint32_t w[4] = {r.x, r.y, r.z, r.w};
+// V neighbouring elements of a row as one access.
+template <typename T, int V> struct alignas(sizeof(T) * V > 16 ? 16 : sizeof(T) * V) Raw {
+    T t[V];
+    __device__ __forceinline__ void load(const T* p) { *this = *reinterpret_cast<const Raw*>(p); }
+    __device__ __forceinline__ void clear() {
 #pragma unroll
-        for (int i = 0; i < 4; ++i) { o[2 * i] = __uint_as_float(w[i] << 16); o[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u); }
+        for (int e = 0; e < V; ++e) t[e] = T(0.f);
+    }
+    __device__ __forceinline__ void get(float* o) const {
+#pragma unroll
+        for (int e = 0; e < V; ++e) o[e] = ldf(t + e);
     }
 };
-template <> struct Raw8<float> {
-    float4 a, b;
-    __device__ __forceinline__ void load(const float* p) { a = reinterpret_cast<const float4*>(p)[0]; b = reinterpret_cast<const float4*>(p)[1]; }
-    __device__ __forceinline__ void clear() { a = b = make_float4(0.f, 0.f, 0.f, 0.f); }
-    __device__ __forceinline__ void get(float* o) const {
-        o[0] = a.x; o[1] = a.y; o[2] = a.z; o[3] = a.w; o[4] = b.x; o[5] = b.y; o[6] = b.z; o[7] = b.w;
-    }
-};
-__device__ __forceinline__ void store8(float* p, const float* v) {
-    reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
-    reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
-}
-__device__ __forceinline__ void store8(__nv_bfloat16* p, const float* v) {
-    uint32_t w[4];
+template <int V, typename T> __device__ __forceinline__ void store(T* p, const float* v) {
+    Raw<T, V> r;
 #pragma unroll
-    for (int i = 0; i < 4; ++i) {
-        const __nv_bfloat162 b = __floats2bfloat162_rn(v[2 * i], v[2 * i + 1]);
-        w[i] = *reinterpret_cast<const uint32_t*>(&b);
-    }
-    *reinterpret_cast<uint4*>(p) = make_uint4(w[0], w[1], w[2], w[3]);
+    for (int e = 0; e < V; ++e) stf(r.t + e, v[e]);
+    *reinterpret_cast<Raw<T, V>*>(p) = r;
 }
 
 // Whether position ``pos`` goes to the cache: in a ring, a row that a later token of the step takes is not written.
@@ -72,21 +60,21 @@ __device__ __forceinline__ bool appended(const ConvQkvArgs& a, int pos, int seq)
     return a.append && !(a.cache.ring_rows && pos < a.kv_len[seq] - a.cache.ring_rows);
 }
 
-template <typename TIn, typename TOut, int TOK>
-__global__ void __launch_bounds__(128) conv_qkv_vec_kernel(ConvQkvArgs a) {
+template <typename TIn, typename TOut, int V, int TOK>
+__global__ void __launch_bounds__(128, V == 4 ? 6 : 3) conv_qkv_vec_kernel(ConvQkvArgs a) {
     pdl_launch_dependents();
-    extern __shared__ float angles[];                 // [TOK][rot/2] cosines, then sines
+    extern __shared__ __align__(16) float angles[];                 // [TOK][rot/2] cosines, then sines
     __shared__ long long row_off[TOK];                // element offset of the token's cache row for kv head 0; < 0: not written
     const int hd = a.hd, C = (a.nh + 2 * a.nkv) * hd, n = a.n_taps, half = a.rope.inv_freq ? a.rope.rot >> 1 : 0;
-    const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * 8, lane = threadIdx.x & 31;
+    const int c0 = (blockIdx.y * blockDim.x + threadIdx.x) * V, lane = threadIdx.x & 31;
     const bool live = c0 < C;                         // (a lane without channels still takes part in the shuffles)
-    float w[NT][8];                                   // the taps depend on nothing that the kernel before makes
+    float w[NT][V];                                   // the taps depend on nothing that the kernel before makes
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
         const int row = j - (NT - n);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) w[j][e] = 0.f;
-        if (live && row >= 0) { Raw8<float> t; t.load(a.taps + (size_t)row * C + c0); t.get(w[j]); }
+        for (int e = 0; e < V; ++e) w[j][e] = 0.f;
+        if (live && row >= 0) { Raw<float, V> t; t.load(a.taps + (size_t)row * C + c0); t.get(w[j]); }
     }
     pdl_wait();
     const int seq = blockIdx.z, first = a.q_start[seq], L = a.q_start[seq + 1] - first, i0 = blockIdx.x * TOK;
@@ -94,8 +82,8 @@ __global__ void __launch_bounds__(128) conv_qkv_vec_kernel(ConvQkvArgs a) {
     const int n_tok = min(TOK, L - i0), slot = a.slot_of_seq[seq], pos0 = a.start_pos[seq] + i0;
     const TIn* in = (const TIn*)a.in + (size_t)first * a.in_stride + c0;
     float* state = a.state ? a.state + (size_t)slot * a.state_stride + c0 : nullptr;
-    Raw8<TIn> raw[TOK];
-    float past[NT - 1][8];                            // rows i0 - 3 .. i0 - 1
+    Raw<TIn, V> raw[TOK];
+    float past[NT - 1][V];                            // rows i0 - 3 .. i0 - 1
 #pragma unroll
     for (int j = 0; j < TOK; ++j) {
         raw[j].clear();
@@ -105,9 +93,9 @@ __global__ void __launch_bounds__(128) conv_qkv_vec_kernel(ConvQkvArgs a) {
     for (int k = 0; k < NT - 1; ++k) {
         const int r = i0 - (NT - 1) + k, old = n - 1 + r;      // row of the step, or (negative) of the state
 #pragma unroll
-        for (int e = 0; e < 8; ++e) past[k][e] = 0.f;
-        if (live && r >= 0) { Raw8<TIn> t; t.load(in + (size_t)r * a.in_stride); t.get(past[k]); }
-        if (live && r < 0 && old >= 0 && state) { Raw8<float> t; t.load(state + (size_t)old * C); t.get(past[k]); }
+        for (int e = 0; e < V; ++e) past[k][e] = 0.f;
+        if (live && r >= 0) { Raw<TIn, V> t; t.load(in + (size_t)r * a.in_stride); t.get(past[k]); }
+        if (live && r < 0 && old >= 0 && state) { Raw<float, V> t; t.load(state + (size_t)old * C); t.get(past[k]); }
     }
     float* cs = angles;
     float* sn = angles + TOK * half;
@@ -122,63 +110,58 @@ __global__ void __launch_bounds__(128) conv_qkv_vec_kernel(ConvQkvArgs a) {
 #pragma unroll
         for (int k = 0; k < NT - 1; ++k) {
             const int idx = L - (NT - 1) + k, row = k - (NT - n);
-            float v[8];
-            if (row >= 0 && idx >= 0) { Raw8<TIn> t; t.load(in + (size_t)idx * a.in_stride); t.get(v); }
+            float v[V];
+            if (row >= 0 && idx >= 0) { Raw<TIn, V> t; t.load(in + (size_t)idx * a.in_stride); t.get(v); }
             // where the step brought fewer, old rows move up: row ``row + L``, which is still as it was
-            if (row >= 0 && idx < 0) { Raw8<float> t; t.load(state + (size_t)(row + L) * C); t.get(v); }
-            if (row >= 0) store8(state + (size_t)row * C, v);
+            if (row >= 0 && idx < 0) { Raw<float, V> t; t.load(state + (size_t)(row + L) * C); t.get(v); }
+            if (row >= 0) store<V>(state + (size_t)row * C, v);
         }
     }
     if (a.zero_in && live) {                          // one token: this thread has read its channels
-        const float z[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-        store8((TIn*)const_cast<void*>(a.in) + (size_t)first * a.in_stride + c0, z);
+        float z[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) z[e] = 0.f;
+        store<V>((TIn*)const_cast<void*>(a.in) + (size_t)first * a.in_stride + c0, z);
     }
     __syncthreads();
     const int head = c0 / hd, e0 = c0 - head * hd;
     const bool is_q = head < a.nh, is_k = !is_q && head < a.nh + a.nkv;
     const bool turns = live && (is_q || is_k) && e0 < 2 * half;
     const bool lower = e0 < half;
-    const int hop = half >> 3, source = a.rope.adjacent || !turns ? lane : (lower ? lane + hop : lane - hop);
-    const size_t head_stride = (size_t)a.cache.page_size * a.cache.head_dim;
+    const int hop = half / V, source = !turns ? lane : (lower ? lane + hop : lane - hop);
+    const bool warp_turns = __any_sync(0xffffffffu, turns);
+    // where this thread's channels go: a query row, or a key or value row beside the cache (if asked) and the cache's own
+    TOut* beside = is_q ? (TOut*)a.q_out + (size_t)(first + i0) * a.q_stride + c0
+                        : (a.kv_out ? (TOut*)a.kv_out + (size_t)(first + i0) * a.kv_stride + (c0 - a.nh * hd) : nullptr);
+    const size_t beside_stride = is_q ? a.q_stride : a.kv_stride;
+    TOut* cached = nullptr;
+    if (!is_q && a.append)
+        cached = (TOut*)a.cache.storage + e0 + (is_k ? 0 : kv_half_elems(a.cache)) + (size_t)(head - a.nh - (is_k ? 0 : a.nkv)) * a.cache.page_size * a.cache.head_dim;
+    const float* trig = angles + (lower ? e0 : e0 - half);
 #pragma unroll
     for (int j = 0; j < TOK; ++j) {
-        float cur[8], y[8];
+        float cur[V], y[V];
         raw[j].get(cur);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) y[e] = fmaf(w[0][e], past[0][e], fmaf(w[1][e], past[1][e], fmaf(w[2][e], past[2][e], w[3][e] * cur[e])));
+        for (int e = 0; e < V; ++e) y[e] = fmaf(w[0][e], past[0][e], fmaf(w[1][e], past[1][e], fmaf(w[2][e], past[2][e], w[3][e] * cur[e])));
 #pragma unroll
-        for (int e = 0; e < 8; ++e) { past[0][e] = past[1][e]; past[1][e] = past[2][e]; past[2][e] = cur[e]; }
-        if (half) {
-            float other[8];
+        for (int e = 0; e < V; ++e) { past[0][e] = past[1][e]; past[1][e] = past[2][e]; past[2][e] = cur[e]; }
+        if (warp_turns) {
+            float other[V];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) other[e] = __shfl_sync(0xffffffffu, y[e], source);
+            for (int e = 0; e < V; ++e) other[e] = __shfl_sync(0xffffffffu, y[e], source);
             if (turns && j < n_tok) {
-                const float* c = cs + j * half;
-                const float* s = sn + j * half;
-                if (a.rope.adjacent) {
+                Raw<float, 4> c[V / 4], sv[V / 4];        // ``half`` is a multiple of V: whole 16 bytes
 #pragma unroll
-                    for (int e = 0; e < 8; e += 2) {
-                        if (e0 + e >= 2 * half) continue;
-                        const int k = (e0 + e) >> 1;
-                        const float u = y[e], v = y[e + 1];
-                        y[e] = u * c[k] - v * s[k]; y[e + 1] = v * c[k] + u * s[k];
-                    }
-                } else {
-                    const int k = lower ? e0 : e0 - half;
+                for (int r = 0; r < V / 4; ++r) { c[r].load(trig + j * half + 4 * r); sv[r].load(trig + (TOK + j) * half + 4 * r); }
 #pragma unroll
-                    for (int e = 0; e < 8; ++e) y[e] = y[e] * c[k + e] + (lower ? -other[e] : other[e]) * s[k + e];
-                }
+                for (int e = 0; e < V; ++e) y[e] = fmaf(lower ? -other[e] : other[e], sv[e / 4].t[e % 4], y[e] * c[e / 4].t[e % 4]);
             }
         }
         if (live && j < n_tok) {
-            const size_t t = first + i0 + j;
             const long long off = row_off[j];
-            if (is_q) store8((TOut*)a.q_out + t * a.q_stride + c0, y);
-            if (!is_q && a.kv_out) store8((TOut*)a.kv_out + t * a.kv_stride + (c0 - a.nh * hd), y);
-            if (!is_q && off >= 0) {
-                TOut* dst = (TOut*)a.cache.storage + off + e0;
-                store8(is_k ? dst + (size_t)(head - a.nh) * head_stride : dst + kv_half_elems(a.cache) + (size_t)(head - a.nh - a.nkv) * head_stride, y);
-            }
+            if (beside) store<V>(beside + j * beside_stride, y);
+            if (cached && off >= 0) store<V>(cached + off, y);
         }
     }
 }
@@ -248,23 +231,32 @@ __global__ void __launch_bounds__(128) conv_qkv_kernel(ConvQkvArgs a, int tile) 
 
 bool aligned16(const void* p) { return ((uintptr_t)p & 15) == 0; }
 
-template <typename TIn, typename TOut, int TOK>
+template <typename TIn, typename TOut, int V, int TOK>
 void launch_vec(const ConvQkvArgs& a, int threads, cudaStream_t stream) {
     const int C = (a.nh + 2 * a.nkv) * a.hd, half = a.rope.inv_freq ? a.rope.rot >> 1 : 0;
-    dim3 grid((a.max_new + TOK - 1) / TOK, (C / 8 + threads - 1) / threads, a.B);
-    tb_launch(conv_qkv_vec_kernel<TIn, TOut, TOK>, grid, dim3(threads), (size_t)2 * TOK * half * sizeof(float), stream, a);
+    dim3 grid((a.max_new + TOK - 1) / TOK, (C / V + threads - 1) / threads, a.B);
+    tb_launch(conv_qkv_vec_kernel<TIn, TOut, V, TOK>, grid, dim3(threads), (size_t)2 * TOK * half * sizeof(float), stream, a);
+}
+
+// A head's lanes (hd / V of them) divide a warp, and rotation partners are whole vectors apart.
+bool vectors_fit(const ConvQkvArgs& a, int V) {
+    const int half = a.rope.inv_freq ? a.rope.rot >> 1 : 0;
+    return a.hd % V == 0 && a.hd / V <= 32 && 32 % (a.hd / V) == 0 && half % V == 0 && (half == 0 || !a.rope.adjacent);
 }
 
 template <typename TIn, typename TOut>
 int launch(const ConvQkvArgs& a, bool any_size, cudaStream_t stream) {
     const int half = a.rope.inv_freq ? a.rope.rot >> 1 : 0, heads = a.nh + 2 * a.nkv;
-    const bool vec = !any_size && a.n_taps <= NT && a.hd >= 16 && a.hd <= 256 && (a.hd & (a.hd - 1)) == 0 && (half % 8 == 0 || a.rope.adjacent) &&
-                     a.in_stride % 8 == 0 && a.q_stride % 8 == 0 && a.kv_stride % 8 == 0 && a.state_stride % 4 == 0 && aligned16(a.in) && aligned16(a.taps) &&
-                     aligned16(a.state) && aligned16(a.q_out) && aligned16(a.kv_out) && aligned16(a.cache.storage);
-    if (vec) {
-        // single tokens: many small blocks (a warp's channels each); longer runs: eight tokens a block (four where rows are float32)
-        if (a.max_new == 1) launch_vec<TIn, TOut, 1>(a, 32, stream);
-        else launch_vec<TIn, TOut, (sizeof(TIn) == 2 ? 8 : 4)>(a, 128, stream);
+    const bool rows = !any_size && a.n_taps <= NT && a.in_stride % 8 == 0 && a.q_stride % 8 == 0 && a.kv_stride % 8 == 0 && a.state_stride % 4 == 0 && aligned16(a.in) &&
+                      aligned16(a.taps) && aligned16(a.state) && aligned16(a.q_out) && aligned16(a.kv_out) && aligned16(a.cache.storage);
+    if (rows && vectors_fit(a, 4)) {
+        if (a.max_new == 1) launch_vec<TIn, TOut, 4, 1>(a, 32, stream);        // single tokens: many small blocks, a warp's channels each
+        else launch_vec<TIn, TOut, 4, RUN>(a, RUN_THREADS, stream);
+        return 0;
+    }
+    if (rows && vectors_fit(a, 8)) {                                           // heads of 256
+        if (a.max_new == 1) launch_vec<TIn, TOut, 8, 1>(a, 32, stream);
+        else launch_vec<TIn, TOut, 8, 4>(a, 128, stream);
         return 0;
     }
     const int tile = a.n_taps - 1 > 8 ? a.n_taps - 1 : 8;
