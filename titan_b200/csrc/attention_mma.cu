@@ -725,13 +725,13 @@ static int launch_decode(const CUtensorMap& map, const DecArgs& d, dim3 grid, cu
 }
 // The largest cluster of this kernel that the device can place: 16 where the non-portable size is allowed
 // and fits (B200), else 8, else 1 (no clusters).
-template <int HD, bool WIDE>
+template <int HD, bool WIDE, bool EXACT = false>
 static int cluster_limit() {
     static int limit = -1;
     if (limit < 0) {
         limit = 1;
         constexpr size_t smem = decode_smem<HD>();
-        auto kernel = attn_decode_mma_kernel<HD, WIDE, true>;
+        auto kernel = attn_decode_mma_kernel<HD, WIDE, true, false, EXACT>;
         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         cudaFuncSetAttribute(kernel, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
         for (int size : {16, 8}) {
@@ -751,10 +751,11 @@ static int cluster_limit() {
 // Launches the kernel; *merged says whether the splits merged among themselves (a cluster) or left their parts in scratch.
 template <int HD, bool WIDE>
 static int launch_decode_any(const CUtensorMap& map, const DecArgs& d, dim3 grid, bool may_cluster, bool exact, bool* merged, cudaStream_t stream) {
-    if (exact) {                     // parts in scratch: the merge kernel finishes
-        *merged = false;
-        TB_REQUIRE(d.scratch && !d.acc, "attn_decode_mma: exact weights leave their parts in scratch memory");
-        return launch_decode<HD, WIDE, false, false, true>(map, d, grid, stream);
+    if (exact) {
+        *merged = may_cluster && (int)grid.z <= cluster_limit<HD, WIDE, true>();
+        TB_REQUIRE(!d.acc, "attn_decode_mma: exact weights come with the head norm as a kernel of its own");
+        TB_REQUIRE(*merged || d.scratch, "attn_decode_mma: %d splits need scratch memory", (int)grid.z);
+        return *merged ? launch_decode<HD, WIDE, true, false, true>(map, d, grid, stream) : launch_decode<HD, WIDE, false, false, true>(map, d, grid, stream);
     }
     *merged = may_cluster && (int)grid.z <= cluster_limit<HD, WIDE>();
     if (d.acc) {
