@@ -54,7 +54,7 @@ CASES = {
                            layer(attention(9, 1, 60, 48, 0.13, 2, 48, 2000.0, (2.0, 1.0, 8.0, 100)), dense(64))],
                           width=136, vocab=211, eps=1e-6, loop=(0, 2, 2)),
     # the whole model runs twice; one expert a token, half of them, all but one
-    "routed": lambda: model([layer(attention(4, 1, 64, 40, 0.125, 4, 16, 10000.0), moe(6, 1, 48, 40)),
+    "routed": lambda: model([layer(attention(3, 1, 64, 40, 0.13, 3, 24, 10000.0), moe(6, 1, 48, 40)),
                              layer(attention(4, 2, 32, 64, 0.18, 2, 32, 700.0, (16.0, 1.0, 3.0, 90)), moe(8, 4, 32)),
                              layer(attention(2, 1, 16, 16, 0.25, 3, 8, 100.0), moe(4, 3, 64, 72))],
                             width=64, vocab=150, eps=1e-5, loop=(0, 3, 2)),

@@ -140,7 +140,7 @@ ATTENTION_SIZES = [
     (9, 1, 60, 48, 2, 48),                  # padded to 64, nine heads on a kv head
     (2, 2, 128, 100, 3, 128),
     (4, 1, 100, 128, 4, 64),                # keys padded to 128
-    (18, 1, 64, 32, 4, 16),                 # more heads on a kv head than the tensor-core decode kernel takes
+    (18, 1, 64, 40, 4, 24),                 # more heads on a kv head than the tensor-core decode kernel takes
     (2, 1, 40, 80, 2, 24),                  # heads of 80
     (2, 1, 200, 256, 3, 96),                # heads of 256
 ]
